@@ -1,4 +1,4 @@
-"""Continuous batching over the captured steps of ``Qwen3DecodeRunner``.
+"""Continuous batching over the captured steps of a ``PagedStepRunner`` (any registered model).
 
 The small serving loop that the hot path needs around it (reference: engine/serving/chunked_prefill.py -
 ``ChunkedPrefillPagedRunner``: admission while a slot and enough pages for the request's full length are free
@@ -29,7 +29,7 @@ from dataclasses import dataclass, field
 
 import torch
 
-from .qwen3_decode import Qwen3DecodeRunner
+from .step_runner import PagedStepRunner
 
 
 class PagePoolExhausted(RuntimeError):
@@ -97,7 +97,7 @@ class ContinuousBatcher:
     different times.  ``step()`` runs one iteration and returns the ``(request id, token)`` pairs it produced;
     ``run()`` drains everything and returns each request's tokens."""
 
-    def __init__(self, runner: Qwen3DecodeRunner, *, max_prefill_tokens: int = 512, mixed: bool = False,
+    def __init__(self, runner: PagedStepRunner, *, max_prefill_tokens: int = 512, mixed: bool = False,
                  use_graphs: bool = True, prefix_cache: bool = False) -> None:
         if max_prefill_tokens < 1:
             raise ValueError("max_prefill_tokens must be positive")
