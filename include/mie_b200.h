@@ -44,6 +44,7 @@ extern "C" {
 #define MIE_STATUS_MAX_LENGTH 32     /* attention read length beyond max_sequence_length */
 #define MIE_STATUS_CAPACITY 64       /* work plan did not fit the scratch the caller sized */
 #define MIE_STATUS_NO_TOKEN 128      /* greedy sampling saw no candidate for a row; token 0 was written */
+#define MIE_STATUS_BAD_TOKEN 256     /* token id outside the vocabulary (row 0 was used) */
 
 /* Element types of K/V pages, queries and activations. */
 #define MIE_DTYPE_BF16 0
@@ -468,6 +469,84 @@ int mie_tp_reduce_rms_norm(const mie_tp_peers_t* peers, int32_t tp, int32_t rank
                            const void* residual, void* summed, const void* weight, int64_t ldq, int32_t scale_ld,
                            int32_t rows, int32_t cols, float eps, uint32_t* state, uint32_t max_polls,
                            int32_t* status, void* stream);
+
+/* ------------------------------------------------------------------------
+ * Decoders with a 32-bit residual stream (no counterpart in the reference)
+ *
+ * Activations (GEMM operands and results, K/V pages, tables and weights named
+ * "T" below) are bf16 or fp32 as `dtype` says; the residual stream, norms,
+ * angles, gates and softmax are fp32.  Sizes are free; rows whose widths,
+ * strides and addresses allow it are moved in vectors.
+ * ---------------------------------------------------------------------- */
+
+/*
+ * x[t] = table[ids[t]] * scale + bigram[row] + sinusoid(positions[t]), stored
+ * as fp32 (out32) and optionally as T (out); every part but the first is
+ * optional.
+ *   bigram [buckets + 1, width] T: row = (previous id * mul_prev + id *
+ *     mul_cur) mod buckets, and row `buckets` at position 0.  The previous id
+ *     is ids[t - 1] when that token is the same sequence's preceding position,
+ *     otherwise it is read from `history`.
+ *   history [num_blocks, block_size] int32: token ids by page slot, one more
+ *     paged cache tensor under the same block tables; every call stores its
+ *     own ids there.
+ *   frequencies [ceil(width / 2)] float64: entries 2i / 2i + 1 get sin / cos of
+ *     positions[t] * frequencies[i].
+ * token_to_sequence may be NULL (token t is block-table row t).
+ */
+int mie_embed_tokens(mie_index_t ids, const void* table, int64_t vocab, float scale, const void* bigram,
+                     int64_t buckets, int64_t mul_prev, int64_t mul_cur, const double* frequencies,
+                     int32_t* history, mie_index_t positions, mie_index_t token_to_sequence,
+                     mie_index_t block_tables, float* out32, void* out, int32_t tokens, int32_t width,
+                     int32_t dtype, int32_t block_size, int32_t num_blocks, int32_t table_rows,
+                     int32_t table_width, int32_t* status, void* stream);
+
+/*
+ * s = alpha * x + y (x fp32, y T or NULL), n = s / sqrt(mean(s^2) + eps),
+ * result n * (weight_offset + weight) with weight T; stored as fp32 (out32,
+ * may be x itself) and / or as T (out).  weight_offset 1 takes weights that are
+ * stored as their deviation from one.
+ */
+int mie_sum_rms_norm(const float* x, int64_t ldx, const void* y, int64_t ldy, float alpha, const void* weight,
+                     float weight_offset, float* out32, int64_t ld32, void* out, int64_t ldo, int32_t rows,
+                     int32_t cols, int32_t dtype, float eps, void* stream);
+
+/*
+ * One pass over a merged projection row [q heads x dim | k heads x dim | v
+ * heads x value_dim] (row stride ld): q and k heads divided by their root mean
+ * square (unit_norm; eps under the root), q times 1 + temp_coef *
+ * ln(floor((position + 1) / temp_every) + 1) (temp_every 0: no temperature),
+ * v <- (1 - lambda) v + lambda v_first (v_first [tokens, kv_heads x value_dim],
+ * row stride ld_first, NULL: none); q to q_out [tokens, q_heads, dim], k and v
+ * to their page slots (last dimension contiguous, other strides free).
+ */
+int mie_qkv_norm_mix_write(const void* qkv, int64_t ld, const void* v_first, int64_t ld_first, float lambda,
+                           int32_t unit_norm, float eps, float temp_coef, int64_t temp_every,
+                           mie_index_t positions, mie_index_t token_to_sequence, mie_index_t block_tables,
+                           void* q_out, mie_view4_t key_blocks, mie_view4_t value_blocks, int32_t tokens,
+                           int32_t q_heads, int32_t kv_heads, int32_t dim, int32_t value_dim, int32_t dtype,
+                           int32_t block_size, int32_t num_blocks, int32_t table_rows, int32_t table_width,
+                           int32_t* status, void* stream);
+
+/* out = g * sigmoid(slope * g) * (u + up_offset), g = min(gate, limit), u = clamp(up, -limit, limit). */
+int mie_clamped_glu(const void* gate, const void* up, int64_t ld_in, void* out, int64_t ldo, int32_t rows,
+                    int32_t cols, int32_t dtype, float limit, float slope, float up_offset, void* stream);
+
+/*
+ * Causal attention of independent rows over K/V pages: row t (position
+ * positions[t], block-table row token_to_sequence[t], or t when that is NULL)
+ * sees the keys j <= position, with window > 0 only the last `window` of them.
+ *   out = sum_j exp(s_j) v_j / (exp(sinks[head]) + sum_j exp(s_j)),
+ *   s_j = (q . k_j) * scale; sinks NULL: no such term.
+ * Any head sizes (dim <= 2048) and page size, bf16 or fp32, fp32 arithmetic.
+ */
+int mie_paged_attention_rows(const void* query, int64_t q_token_stride, int64_t q_head_stride, void* out,
+                             int64_t o_token_stride, int64_t o_head_stride, mie_view4_t key_blocks,
+                             mie_view4_t value_blocks, mie_index_t positions, mie_index_t token_to_sequence,
+                             mie_index_t block_tables, int32_t tokens, int32_t q_heads, int32_t kv_heads,
+                             int32_t dim, int32_t value_dim, int32_t block_size, int32_t num_blocks,
+                             int32_t table_rows, int32_t table_width, int32_t dtype, float scale, int64_t window,
+                             const float* sinks, int32_t* status, void* stream);
 
 #ifdef __cplusplus
 }

@@ -23,6 +23,7 @@ STATUS_WAIT_TIMEOUT = 16
 STATUS_MAX_LENGTH = 32
 STATUS_CAPACITY = 64
 STATUS_NO_TOKEN = 128
+STATUS_BAD_TOKEN = 256
 
 GEMM_NO_WEIGHT_PREFETCH = 1
 
@@ -35,6 +36,7 @@ STATUS_MESSAGES = {
     STATUS_MAX_LENGTH: "max_sequence_length does not cover the attention read length",
     STATUS_CAPACITY: "decode work plan exceeded its scratch capacity",
     STATUS_NO_TOKEN: "greedy sampling found no candidate for a row (token 0 was substituted)",
+    STATUS_BAD_TOKEN: "a token id lies outside the vocabulary",
 }
 
 DTYPE_CODES = {torch.bfloat16: 0, torch.float16: 1, torch.float32: 2}
@@ -125,6 +127,21 @@ _SIGNATURES: dict[str, tuple[object, list[object]]] = {
     "mie_tp_reduce_rms_norm": (ctypes.c_int, [ctypes.POINTER(TpPeersT), c_int32, c_int32, c_int64, c_void_p, c_void_p,
                                               c_void_p, c_int64, c_int32, c_int32, c_int32, c_float, c_void_p,
                                               ctypes.c_uint32, c_void_p, c_void_p]),
+    "mie_embed_tokens": (ctypes.c_int, [IndexT, c_void_p, c_int64, c_float, c_void_p, c_int64, c_int64, c_int64,
+                                        c_void_p, c_void_p, IndexT, IndexT, IndexT, c_void_p, c_void_p, c_int32,
+                                        c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
+    "mie_sum_rms_norm": (ctypes.c_int, [c_void_p, c_int64, c_void_p, c_int64, c_float, c_void_p, c_float, c_void_p,
+                                        c_int64, c_void_p, c_int64, c_int32, c_int32, c_int32, c_float, c_void_p]),
+    "mie_qkv_norm_mix_write": (ctypes.c_int, [c_void_p, c_int64, c_void_p, c_int64, c_float, c_int32, c_float,
+                                              c_float, c_int64, IndexT, IndexT, IndexT, c_void_p, View4T, View4T,
+                                              c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                              c_int32, c_int32, c_void_p, c_void_p]),
+    "mie_clamped_glu": (ctypes.c_int, [c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int32, c_int32, c_int32,
+                                       c_float, c_float, c_float, c_void_p]),
+    "mie_paged_attention_rows": (ctypes.c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, View4T,
+                                                View4T, IndexT, IndexT, IndexT, c_int32, c_int32, c_int32, c_int32,
+                                                c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_float,
+                                                c_int64, c_void_p, c_void_p, c_void_p]),
 }
 
 _lib: ctypes.CDLL | None = None

@@ -8,6 +8,7 @@ mini_inference_engine_b200.build`` rebuilds when a source changed.
 
 from __future__ import annotations
 
+import fcntl
 import hashlib
 import os
 import shutil
@@ -61,8 +62,14 @@ def build_library(force: bool = False, verbose: bool = False) -> Path:
 
     if not force and is_current():
         return LIB_PATH
-    nvcc = _nvcc()
     OBJ_DIR.mkdir(exist_ok=True)
+    with open(OBJ_DIR / "lock", "w") as lock:  # one builder at a time; the others find its result
+        fcntl.flock(lock, fcntl.LOCK_EX)
+        return LIB_PATH if not force and is_current() else _compile(verbose)
+
+
+def _compile(verbose: bool) -> Path:
+    nvcc = _nvcc()
     log_dir = OBJ_DIR
 
     def compile_one(src: Path) -> Path:
@@ -78,10 +85,12 @@ def build_library(force: bool = False, verbose: bool = False) -> Path:
 
     with ThreadPoolExecutor(max_workers=min(8, os.cpu_count() or 1)) as pool:
         objects = list(pool.map(compile_one, _sources()))
-    link = [nvcc, "-shared", "-o", str(LIB_PATH), *map(str, objects)]
+    fresh = LIB_PATH.with_suffix(".so.new")
+    link = [nvcc, "-shared", "-o", str(fresh), *map(str, objects)]
     done = subprocess.run(link, capture_output=True, text=True)
     if done.returncode != 0:
         raise RuntimeError(f"link failed:\n{done.stdout}\n{done.stderr}")
+    os.replace(fresh, LIB_PATH)
     STAMP_PATH.write_text(source_digest())
     return LIB_PATH
 

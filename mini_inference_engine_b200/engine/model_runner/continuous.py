@@ -27,9 +27,7 @@ from __future__ import annotations
 from collections import OrderedDict, deque
 from dataclasses import dataclass, field
 
-import torch
-
-from .step_runner import PagedStepRunner
+from .step_runner import PagedStepRunner, eager_step
 
 
 class PagePoolExhausted(RuntimeError):
@@ -300,57 +298,15 @@ class ContinuousBatcher:
             record["h2d_bytes"] = h2d
             record["bucket"] = next(b for b in runner.decode_buckets if b >= len(decoding))
             return tokens
-        device = runner.device
-        width = runner.table_width
-        tables = torch.full((len(decoding), width), -1, dtype=torch.int32)
-        for row, pages in enumerate(blocks):
-            tables[row, :len(pages)] = torch.tensor(pages, dtype=torch.int32)
-        out = runner.decode_forward(torch.tensor(ids, dtype=torch.int64, device=device),
-                                    torch.tensor(lengths, dtype=torch.int32, device=device), tables.to(device))
-        return out.tolist()
+        return eager_step(runner, ids, lengths, blocks, []).tolist()
 
     def _prefill(self, chunk_items) -> list[int]:
-        runner, device = self.runner, self.runner.device
-        width = runner.table_width
-        counts = [len(tokens) for tokens, _, _ in chunk_items]
-        flat = torch.tensor([t for tokens, _, _ in chunk_items for t in tokens], dtype=torch.int64, device=device)
-        tok2seq = torch.cat([torch.full((n,), i, dtype=torch.int32) for i, n in enumerate(counts)]).to(device)
-        tokpos = torch.cat([torch.arange(start, start + n, dtype=torch.int32)
-                            for (_, start, _), n in zip(chunk_items, counts)]).to(device)
-        tables = torch.full((len(chunk_items), width), -1, dtype=torch.int32)
-        for row, (_, _, pages) in enumerate(chunk_items):
-            tables[row, :len(pages)] = torch.tensor(pages, dtype=torch.int32)
-        cu = torch.zeros(len(counts) + 1, dtype=torch.int32)
-        cu[1:] = torch.tensor(counts, dtype=torch.int32).cumsum(0)
-        kv_lens = torch.tensor([start + n for (_, start, _), n in zip(chunk_items, counts)], dtype=torch.int32)
-        out = runner.prefill_forward(flat, tok2seq, tokpos, tables.to(device), cu.to(device), kv_lens.to(device),
-                                     max(counts))
-        return out.tolist()
+        return eager_step(self.runner, [], [], [], chunk_items).tolist()
 
     def _mixed(self, ids, lengths, blocks, chunk_items) -> tuple[list[int], list[int]]:
-        runner = self.runner
         if self.use_graphs:
-            return runner.mixed_rows(ids, lengths, blocks, chunk_items)
-        device, width = runner.device, runner.table_width
-        live, counts = len(ids), [len(tokens) for tokens, _, _ in chunk_items]
-        flat = torch.tensor(list(ids) + [t for tokens, _, _ in chunk_items for t in tokens], dtype=torch.int64)
-        tok2seq = torch.cat([torch.arange(live, dtype=torch.int32),
-                             *[torch.full((n,), live + i, dtype=torch.int32) for i, n in enumerate(counts)]])
-        tokpos = torch.cat([torch.tensor(lengths, dtype=torch.int32) - 1,
-                            *[torch.arange(start, start + n, dtype=torch.int32)
-                              for (_, start, _), n in zip(chunk_items, counts)]])
-        tables = torch.full((live + len(chunk_items), width), -1, dtype=torch.int32)
-        for row, pages in enumerate(list(blocks) + [pages for _, _, pages in chunk_items]):
-            tables[row, :len(pages)] = torch.tensor(pages, dtype=torch.int32)
-        cu = torch.zeros(len(counts) + 1, dtype=torch.int32)
-        cu[1:] = torch.tensor(counts, dtype=torch.int32).cumsum(0)
-        kv_lens = torch.tensor([start + n for (_, start, _), n in zip(chunk_items, counts)], dtype=torch.int32)
-        logit_rows = torch.cat([torch.arange(live, dtype=torch.int64), live + cu[1:].long() - 1])
-        out = runner.mixed_forward(flat.to(device), tok2seq.to(device), tokpos.to(device), tables.to(device),
-                                   decode_rows=live,
-                                   decode_lengths=torch.tensor(lengths, dtype=torch.int32, device=device) if live else None,
-                                   cu_seqlens=cu.to(device), kv_lens=kv_lens.to(device), max_query_len=max(counts),
-                                   logit_rows=logit_rows.to(device)).tolist()
+            return self.runner.mixed_rows(ids, lengths, blocks, chunk_items)
+        out, live = eager_step(self.runner, ids, lengths, blocks, chunk_items).tolist(), len(ids)
         return out[:live], out[live:]
 
     def run(self, max_iterations: int = 100000) -> dict[object, list[int]]:

@@ -323,9 +323,8 @@ class Qwen3DecodeRunner(PagedStepRunner):
         self.scratch = decode_scratch(max(max_batch, self.decode_buckets[-1]), self.local_q_heads,
                                       self.local_kv_heads, shape.head_dim, max_batch * max_context, self.device)
         # lm_head + greedy sampling: one pass over the tied embedding that never writes the logits
-        # (mie_lm_head_argmax) unless MIE_LM_HEAD=cublas; its per-row keys are zero between calls.
+        # (mie_lm_head_argmax) unless MIE_LM_HEAD=cublas.
         self.fused_lm_head = os.environ.get("MIE_LM_HEAD", "fused") != "cublas"
-        self._lm_keys = torch.zeros(256, dtype=torch.int64, device=self.device)
         # Tensor parallel decode: the all-reduce after o_proj / down_proj is fused into the residual add +
         # RMSNorm + quantisation kernel over peer memory unless MIE_TP_EXCHANGE=nccl (or fused_exchange=False).
         if fused_exchange is None:
@@ -487,17 +486,8 @@ class Qwen3DecodeRunner(PagedStepRunner):
         """Greedy next tokens of normed hidden rows ``[rows, hidden]`` (rows <= 256): the bf16 product with the
         tied lm_head and its argmax in one pass (reference: engine/model_runner/qwen3_mixed.py:164-174)."""
 
-        lib = _lib.load()
-        rows = int(final.shape[0])
-        if final.stride(1) != 1 or final.stride(0) % 8 != 0 or final.data_ptr() % 16 != 0:
-            final = final.contiguous()
-        head = self.weights.lm_head
-        tokens = torch.empty(rows, dtype=torch.int64, device=self.device)
-        values = torch.empty(rows, dtype=torch.int32, device=self.device) if self.tp > 1 else None
-        _lib.check(lib.mie_lm_head_argmax(_lib.ptr(final), final.stride(0), _lib.ptr(head), head.stride(0), rows,
-                                          head.shape[0], head.shape[1], self.weights.vocab_start,
-                                          _lib.ptr(self._lm_keys), _lib.ptr(tokens), _lib.ptr(values),
-                                          _lib.ptr(self.status), _lib.stream_arg(self.device)))
+        values = torch.empty(final.shape[0], dtype=torch.int32, device=self.device) if self.tp > 1 else None
+        tokens = self.lm_head_argmax(final, self.weights.lm_head, self.weights.vocab_start, values)
         return sharded_greedy_from_pairs(tokens, values, self.tp, self.group) if self.tp > 1 else tokens
 
     # -- flat forward: decode rows and packed prompt chunks in one token stream --------------------------

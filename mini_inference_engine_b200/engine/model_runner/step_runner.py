@@ -14,6 +14,7 @@ import torch
 from ... import _lib
 
 
+LM_HEAD_MAX_ROWS = 256  # rows one mie_lm_head_argmax call takes
 DEFAULT_DECODE_BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 256)
 
 
@@ -258,6 +259,45 @@ class MixedBuffers:
         return copied
 
 
+def eager_step(runner, decode_ids, decode_lengths, decode_blocks, chunks, *, logit_rows=None,
+               return_logits: bool = False):
+    """One step of a runner from host data without a graph.  ``decode_*``: one token per row (id, length
+    including it, page ids); ``chunks``: ``(token ids, start position, page ids)``.  The flat stream is the
+    decode rows followed by the chunks; ``logit_rows`` picks rows of it (default: every decode row and each
+    chunk's last row).  Returns what the forward returns for those rows."""
+
+    device, live = runner.device, len(decode_ids)
+    extra = {"return_logits": True} if return_logits else {}
+    counts = [len(tokens) for tokens, _, _ in chunks]
+    tables = torch.full((live + len(chunks), runner.table_width), -1, dtype=torch.int32)
+    for row, pages in enumerate([*decode_blocks, *(pages for _, _, pages in chunks)]):
+        tables[row, :len(pages)] = torch.tensor(pages, dtype=torch.int32)
+    tables = tables.to(device)
+    lengths = torch.tensor(decode_lengths, dtype=torch.int32)
+    if not chunks and (logit_rows is None or list(logit_rows) == list(range(live))):
+        return runner.decode_forward(torch.tensor(decode_ids, dtype=torch.int64, device=device), lengths.to(device),
+                                     tables, **extra)
+    flat = torch.tensor([*decode_ids, *(t for tokens, _, _ in chunks for t in tokens)], dtype=torch.int64).to(device)
+    tok2seq = torch.cat([torch.arange(live, dtype=torch.int32),
+                         *[torch.full((n,), live + i, dtype=torch.int32) for i, n in enumerate(counts)]]).to(device)
+    tokpos = torch.cat([lengths - 1, *[torch.arange(start, start + n, dtype=torch.int32)
+                                       for (_, start, _), n in zip(chunks, counts)]]).to(device)
+    cu = torch.zeros(len(counts) + 1, dtype=torch.int32)
+    if counts:
+        cu[1:] = torch.tensor(counts, dtype=torch.int32).cumsum(0)
+    kv_lens = torch.tensor([start + n for (_, start, _), n in zip(chunks, counts)], dtype=torch.int32).to(device)
+    longest = max(counts, default=0)
+    if not live and logit_rows is None:
+        return runner.prefill_forward(flat, tok2seq, tokpos, tables, cu.to(device), kv_lens, longest, **extra)
+    if logit_rows is None:
+        rows = torch.cat([torch.arange(live, dtype=torch.int64), live + cu[1:].long() - 1])
+    else:
+        rows = torch.tensor(logit_rows, dtype=torch.int64)
+    return runner.mixed_forward(flat, tok2seq, tokpos, tables, decode_rows=live,
+                                decode_lengths=lengths.to(device) if live else None, cu_seqlens=cu.to(device),
+                                kv_lens=kv_lens, max_query_len=longest, logit_rows=rows.to(device), **extra)
+
+
 class PagedStepRunner:
     """Steps over paged per-request state: decode rows, packed prompt chunks or both in one flat forward, eager
     or replayed from CUDA graphs captured per bucket.
@@ -293,6 +333,31 @@ class PagedStepRunner:
         self._graphs: dict[tuple, tuple[torch.cuda.CUDAGraph, object]] = {}
         self._generation = 0  # distinguishes the rows of successive generate() calls
         self.launches_per_step = 0
+        self._lm_keys = torch.zeros(LM_HEAD_MAX_ROWS, dtype=torch.int64, device=device)  # zero between calls
+
+    # -- greedy sampling ---------------------------------------------------------------------------
+
+    @staticmethod
+    def can_fuse_lm_head(final: torch.Tensor, head: torch.Tensor) -> bool:
+        """Whether ``lm_head_argmax`` takes these rows: bf16, few enough, a width of whole 16-byte groups."""
+
+        return bool(final.dtype == head.dtype == torch.bfloat16 and final.shape[0] <= LM_HEAD_MAX_ROWS
+                    and head.shape[1] % 8 == 0 and head.stride(0) % 8 == 0 and head.data_ptr() % 16 == 0)
+
+    def lm_head_argmax(self, final: torch.Tensor, head: torch.Tensor, vocab_start: int = 0,
+                       values: torch.Tensor | None = None) -> torch.Tensor:
+        """Greedy next tokens of normed hidden rows: the bf16 product with the head and its argmax in one pass
+        over the vocabulary that never writes the logits (``mie_lm_head_argmax``)."""
+
+        rows = int(final.shape[0])
+        if final.stride(1) != 1 or final.stride(0) % 8 != 0 or final.data_ptr() % 16 != 0:
+            final = final.contiguous()
+        tokens = torch.empty(rows, dtype=torch.int64, device=self.device)
+        _lib.check(_lib.load().mie_lm_head_argmax(
+            _lib.ptr(final), final.stride(0), _lib.ptr(head), head.stride(0), rows, head.shape[0], head.shape[1],
+            vocab_start, _lib.ptr(self._lm_keys), _lib.ptr(tokens), _lib.ptr(values), _lib.ptr(self.status),
+            _lib.stream_arg(self.device)))
+        return tokens
 
     # -- the two forwards of a model -------------------------------------------------------------
 
@@ -492,4 +557,5 @@ class PagedStepRunner:
         _lib.raise_for_status(self.status)
 
 
-__all__ = ["DEFAULT_DECODE_BUCKETS", "DecodeBuffers", "MixedBuffers", "PADDING", "PagedStepRunner", "select_bucket"]
+__all__ = ["DEFAULT_DECODE_BUCKETS", "DecodeBuffers", "MixedBuffers", "PADDING", "PagedStepRunner", "eager_step",
+           "select_bucket"]
