@@ -548,6 +548,39 @@ int mie_paged_attention_rows(const void* query, int64_t q_token_stride, int64_t 
                              int32_t table_rows, int32_t table_width, int32_t dtype, float scale, int64_t window,
                              const float* sinks, int32_t* status, void* stream);
 
+/*
+ * The same attention on the streaming kernels, bf16 only.  Both see pages
+ * [num_blocks, kv_heads, block_size, dim or value_dim] (last dimension
+ * contiguous, 16-byte aligned rows), head sizes that are multiples of 8, any
+ * GQA group; *_supported (host arithmetic) says whether sizes are taken.
+ *
+ * mie_sink_decode_attention: one query row per request, lengths count it.
+ * Work plan, split_policy, scratch (mie_decode_scratch_bytes with kv_heads and
+ * value_dim), use_plan / plan_slot as in mie_paged_decode_attention; a plan
+ * may be reused by calls with the same sizes, lengths and window.
+ *
+ * mie_sink_prefill_attention: packed chunks, query row i of request r at
+ * position kv_lens[r] - q_len + i, as in mie_flash_prefill_attention.
+ */
+int mie_sink_decode_supported(int32_t dim, int32_t value_dim, int32_t block_size, int32_t dtype);
+int mie_sink_decode_attention(const void* query, int64_t q_row_stride, int64_t q_head_stride, void* out,
+                              int64_t o_row_stride, int64_t o_head_stride, mie_view4_t key_blocks,
+                              mie_view4_t value_blocks, mie_index_t block_tables, mie_index_t sequence_lengths,
+                              int32_t batch, int32_t q_heads, int32_t kv_heads, int32_t dim, int32_t value_dim,
+                              int32_t block_size, int32_t num_blocks, int32_t table_width, int32_t dtype,
+                              float scale, int64_t window, const float* sinks, int32_t split_policy, void* scratch,
+                              int64_t scratch_bytes, int32_t use_plan, int32_t plan_slot, int32_t* status,
+                              void* stream);
+int mie_sink_prefill_supported(int32_t q_heads, int32_t kv_heads, int32_t dim, int32_t value_dim,
+                               int32_t block_size, int32_t dtype, float scale);
+int mie_sink_prefill_attention(const void* query, int64_t q_token_stride, int64_t q_head_stride, void* out,
+                               int64_t o_token_stride, int64_t o_head_stride, mie_view4_t key_blocks,
+                               mie_view4_t value_blocks, mie_index_t block_tables, mie_index_t cu_seqlens,
+                               mie_index_t kv_lens, int32_t requests, int32_t max_query_len, int32_t q_heads,
+                               int32_t kv_heads, int32_t dim, int32_t value_dim, int32_t block_size,
+                               int32_t num_blocks, int32_t table_width, int32_t dtype, float scale, int64_t window,
+                               const float* sinks, int32_t* status, void* stream);
+
 #ifdef __cplusplus
 }
 #endif

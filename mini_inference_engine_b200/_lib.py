@@ -142,6 +142,16 @@ _SIGNATURES: dict[str, tuple[object, list[object]]] = {
                                                 View4T, IndexT, IndexT, IndexT, c_int32, c_int32, c_int32, c_int32,
                                                 c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_float,
                                                 c_int64, c_void_p, c_void_p, c_void_p]),
+    "mie_sink_decode_supported": (ctypes.c_int, [c_int32, c_int32, c_int32, c_int32]),
+    "mie_sink_decode_attention": (ctypes.c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, View4T,
+                                                 View4T, IndexT, IndexT, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                                 c_int32, c_int32, c_int32, c_int32, c_float, c_int64, c_void_p,
+                                                 c_int32, c_void_p, c_int64, c_int32, c_int32, c_void_p, c_void_p]),
+    "mie_sink_prefill_supported": (ctypes.c_int, [c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_float]),
+    "mie_sink_prefill_attention": (ctypes.c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, View4T,
+                                                  View4T, IndexT, IndexT, IndexT, c_int32, c_int32, c_int32, c_int32,
+                                                  c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_float,
+                                                  c_int64, c_void_p, c_void_p, c_void_p]),
 }
 
 _lib: ctypes.CDLL | None = None

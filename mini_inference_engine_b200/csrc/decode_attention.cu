@@ -19,514 +19,10 @@
 #include <mutex>
 #include <unordered_map>
 
-#include "common.cuh"
+#include "decode_attention.cuh"
 
 namespace mie {
 namespace {
-
-constexpr int kWarps = 8;
-constexpr int kStages = 3;
-constexpr int kTileTokens = 16;
-constexpr int kHeadDim = 128;
-constexpr int kTileBytes = kTileTokens * kHeadDim * 2;  // one K or V tile
-constexpr int kStageBytes = 2 * kTileBytes;             // K + V
-constexpr int kPidBatch = 128;                          // tiles whose page ids are staged at once
-constexpr int kMinChunk = 64;
-constexpr int kMaxChunk = 2048;
-constexpr int kPlanThreads = 1024;
-constexpr int kHeaderInts = 128;  // [0]=chunk [1]=seq_chunks [2]=items; [16..79] work counters
-constexpr int kCounterBase = 16;
-constexpr int kCounters = 64;
-constexpr int kMaxGroupMerge = 4;  // query heads per KV head the merge kernel handles in one block
-
-struct View4 {
-  char* ptr;
-  long long s[4];
-  __host__ View4(const mie_view4_t& v) : ptr(reinterpret_cast<char*>(v.ptr)) {
-    for (int i = 0; i < 4; ++i) s[i] = v.stride[i];
-  }
-};
-
-struct Scratch {
-  int* header;
-  int* offsets;     // [batch + 1]
-  int* item_seq;    // [cap]
-  int* item_chunk;  // [cap]
-  float* part_m;    // [cap][q_heads]
-  float* part_l;    // [cap][q_heads]
-  float* part_o;    // [cap][q_heads][head_dim]
-  int cap;
-};
-
-template <typename T>
-__device__ __forceinline__ float round_act(float v) {
-  return to_float<T>(from_float<T>(v));
-}
-
-__host__ __device__ inline long long align_up(long long v, long long a) { return (v + a - 1) / a * a; }
-
-// Attention read length of request b, or 0 (with a status bit) when the
-// metadata is unusable.
-__device__ __forceinline__ long long read_length(const IndexView& lengths, const IndexView& positions, int b,
-                                                 long long capacity, int* status) {
-  const long long len = lengths.at(b);
-  if (len < 1 || len > capacity) {
-    raise_status(status, MIE_STATUS_BAD_LENGTH);
-    return 0;
-  }
-  if (!positions.valid()) return len;
-  const long long pos = positions.at(b);
-  if (pos < 0) {
-    raise_status(status, MIE_STATUS_BAD_POSITION);
-    return 0;
-  }
-  return pos + 1 < len ? pos + 1 : len;
-}
-
-// ---------------------------------------------------------------------------
-// Plan kernel: one CTA.
-// ---------------------------------------------------------------------------
-__device__ __forceinline__ long long block_sum_ll(long long v, long long* smem) {
-  const int lane = threadIdx.x & 31, warp = threadIdx.x >> 5;
-#pragma unroll
-  for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-  if (lane == 0) smem[warp] = v;
-  __syncthreads();
-  long long t = 0;
-  for (int i = 0; i < (int)(blockDim.x >> 5); ++i) t += smem[i];
-  __syncthreads();
-  return t;
-}
-
-// Split-KV planning.  The decode kernel is a dynamic queue of (request, chunk, KV head) items over
-// `warps` persistent warps, so its time is close to
-//     ceil(items / warps) x (time of one chunk + what a warp loses between two items),
-// with items = kv_heads x sum_b ceil(length_b / chunk).  Policy 1 evaluates that with the batch's real
-// lengths for a grid of chunk sizes and takes the cheapest: a chunk size that just misses a whole number of
-// rounds costs a full extra round on a few warps (see the limit below for where this applies).
-// `switch_tokens` is the between-items loss (queue pop,
-// metadata, refilling the TMA ring, writing and later merging a partial) expressed in tokens of streaming;
-// 128 tokens of one bf16 KV head (64 KB) reproduces the measured ranking of chunk sizes on an 8-way
-// head shard (384 and 1024 tokens best, 512 and 192 worst).
-constexpr int kPlanCands = 21;
-// Candidate j (compile-time in the unrolled loops, so the divisions below are by constants).
-__host__ __device__ constexpr int plan_chunk(int j) {
-  constexpr int table[kPlanCands] = {64,  80,  96,  112, 128, 160, 192,  224,  256,  320, 384,
-                                     448, 512, 640, 768, 896, 1024, 1280, 1536, 1792, 2048};
-  return table[j];
-}
-
-__global__ void __launch_bounds__(kPlanThreads) plan_kernel(IndexView lengths, IndexView positions, int batch,
-                                                            long long capacity_tokens, int kv_heads, int policy,
-                                                            int warps, int switch_tokens, Scratch sc, int* status) {
-  __shared__ long long red[32];
-  __shared__ int warp_tot[32];
-  __shared__ int cand_part[32][kPlanCands];
-  __shared__ int cand_count[kPlanCands];
-  __shared__ int running_s;
-  __shared__ long long chunk_s;
-  const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
-  chain_wait();
-  chain_release();
-
-  // With one thread per request (the usual launch) a request's length is read once and kept.
-  const bool one_each = batch <= (int)blockDim.x;
-  long long own = 0, local = 0;
-  if (one_each) {
-    if (tid < batch) own = read_length(lengths, positions, tid, capacity_tokens, status);
-    local = own;
-  } else {
-    for (int b = tid; b < batch; b += blockDim.x) local += read_length(lengths, positions, b, capacity_tokens, status);
-  }
-  const long long total = block_sum_ll(local, red);
-  const long long room = sc.cap - batch;  // > 0, checked on the host
-
-  long long chunk;
-  if (policy == 0) {
-    chunk = (1ll << 40);
-  } else if (policy == 1) {
-    int mine[kPlanCands];
-#pragma unroll
-    for (int j = 0; j < kPlanCands; ++j) mine[j] = 0;
-    for (int b = tid; b < batch; b += blockDim.x) {
-      const int rl = (int)(one_each ? own : read_length(lengths, positions, b, capacity_tokens, nullptr));
-#pragma unroll
-      for (int j = 0; j < kPlanCands; ++j) mine[j] += (rl + plan_chunk(j) - 1) / plan_chunk(j);
-    }
-#pragma unroll
-    for (int j = 0; j < kPlanCands; ++j) {
-      int v = mine[j];
-#pragma unroll
-      for (int o = 16; o > 0; o >>= 1) v += __shfl_xor_sync(0xffffffffu, v, o);
-      if (lane == 0) cand_part[warp][j] = v;
-    }
-    __syncthreads();
-    if (tid < kPlanCands) {
-      int t = 0;
-      for (int w = 0; w < (int)(blockDim.x >> 5); ++w) t += cand_part[w][tid];
-      cand_count[tid] = t;
-    }
-    __syncthreads();
-    if (tid == 0) {
-      // With several KV heads per rank and enough work for four items of at least 512 tokens per warp the kernel is bound by
-      // HBM, not by the queue's rounds, and finer items measured better (C=256 at 1 / 2 ranks): there the
-      // chunk stays at or below the four-items-per-warp size.  A single KV head per rank, or a batch too
-      // small for that, is where whole rounds decide.
-      long long limit = kMaxChunk;
-      if (kv_heads >= 2) {
-        const long long four = align_up((total * kv_heads + 4ll * warps - 1) / (4ll * warps), kTileTokens);
-        if (four >= 512) limit = four;
-      }
-      long long best = plan_chunk(0);
-      long long best_cost = -1;
-#pragma unroll
-      for (int j = kPlanCands - 1; j >= 0; --j) {  // larger chunks first: they win ties (fewer partials)
-        if (plan_chunk(j) > limit && j > 0) continue;
-        if (cand_count[j] > sc.cap) continue;      // more (request, chunk) pairs than the scratch holds
-        const long long items = (long long)cand_count[j] * kv_heads;
-        const long long rounds = (items + warps - 1) / warps;
-        const long long cost = rounds * (plan_chunk(j) + switch_tokens);
-        if (best_cost < 0 || cost < best_cost) {
-          best_cost = cost;
-          best = plan_chunk(j);
-        }
-      }
-      chunk_s = best;
-    }
-    __syncthreads();
-    chunk = chunk_s;
-  } else {
-    chunk = align_up(policy, kTileTokens);
-  }
-  // Never emit more (request, chunk) pairs than the caller's scratch holds.
-  if (total / chunk + batch > sc.cap) {
-    chunk = align_up((total + room - 1) / room, kTileTokens);  // still exact, only coarser
-  }
-
-  // Work list in request order, a request's chunks next to each other (queueing the full-sized chunks of
-  // all requests first and the shorter last chunks at the end was measured 2 % slower at the same chunk size:
-  // neighbouring items then no longer read neighbouring pages).
-  if (tid == 0) running_s = 0;
-  __syncthreads();
-  for (int base = 0; base < batch; base += blockDim.x) {
-    const int b = base + tid;
-    int c = 0;
-    if (b < batch) {
-      const long long rl = one_each ? own : read_length(lengths, positions, b, capacity_tokens, nullptr);
-      c = (int)((rl + chunk - 1) / chunk);
-    }
-    int incl = c;
-#pragma unroll
-    for (int o = 1; o < 32; o <<= 1) {
-      const int n = __shfl_up_sync(0xffffffffu, incl, o);
-      if (lane >= o) incl += n;
-    }
-    if (lane == 31) warp_tot[warp] = incl;
-    __syncthreads();
-    int before = running_s;
-    for (int w = 0; w < warp; ++w) before += warp_tot[w];
-    const int excl = before + incl - c;
-    if (b < batch) {
-      sc.offsets[b] = excl;
-      for (int j = 0; j < c; ++j) {
-        sc.item_seq[excl + j] = b;
-        sc.item_chunk[excl + j] = j;
-      }
-    }
-    __syncthreads();
-    if (tid == 0) {
-      int t = 0;
-      for (int w = 0; w < (int)(blockDim.x >> 5); ++w) t += warp_tot[w];
-      running_s += t;
-    }
-    __syncthreads();
-  }
-  const int pairs = running_s;
-  if (tid == 0) {
-    sc.offsets[batch] = pairs;
-    sc.header[0] = (int)(chunk > 0x7fffffffll ? 0x7fffffff : chunk);
-    sc.header[1] = pairs;
-    sc.header[2] = pairs * kv_heads;
-  }
-  if (tid < kCounters) sc.header[kCounterBase + tid] = 0;
-}
-
-// ---------------------------------------------------------------------------
-// Main kernel
-// ---------------------------------------------------------------------------
-struct DecodeParams {
-  View4 q, out;
-  IndexView tables, lengths, positions;
-  Scratch sc;
-  int batch, q_heads, kv_heads, group, block_size, num_blocks, table_width;
-  float scale_log2;
-  int counter_slot;
-  int* status;
-  uint8_t* out_q8;     // optional e4m3 copy of the output for the next FP8 GEMM: [batch][ldq8 bytes]
-  long long ldq8;
-  float* out_scales;   // [q_heads][out_scale_ld]: one scale per (head, request) = per 128 columns
-  int out_scale_ld;
-  int merge_head0;     // first head of the group handled by this merge launch
-};
-
-template <typename T>
-__global__ void __launch_bounds__(kWarps * 32, 1)
-    decode_kernel(const __grid_constant__ CUtensorMap kmap, const __grid_constant__ CUtensorMap vmap,
-                  const DecodeParams p) {
-  extern __shared__ uint8_t smem_raw[];
-  uint8_t* smem = reinterpret_cast<uint8_t*>(align_up((long long)reinterpret_cast<uintptr_t>(smem_raw), 1024));
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  uint8_t* stages = smem + (size_t)warp * kStages * kStageBytes;
-  uint64_t* bars = reinterpret_cast<uint64_t*>(smem + (size_t)kWarps * kStages * kStageBytes) + warp * kStages;
-  int* pids = reinterpret_cast<int*>(smem + (size_t)kWarps * kStages * kStageBytes + kWarps * kStages * 8) +
-              warp * kPidBatch;
-
-  if (lane == 0) {
-    for (int s = 0; s < kStages; ++s) mbar_init(&bars[s], 1);
-    mbar_fence_init();
-    tma_prefetch_desc(&kmap);
-    tma_prefetch_desc(&vmap);
-  }
-  __syncthreads();
-  chain_wait();
-  chain_release();
-
-  const int g = lane >> 2, t = lane & 3;
-  const int chunk = p.sc.header[0];
-  const int total_items = p.sc.header[2];
-  int* counter = p.sc.header + kCounterBase + p.counter_slot;
-  const long long capacity_tokens = (long long)p.table_width * p.block_size;
-  uint32_t parity = 0;
-  const uint64_t stream_policy = l2_evict_first_policy();  // K/V pages are read once per step
-
-  // ldmatrix lane geometry (constant per lane).
-  const int k_tok = (lane & 7) + ((lane >> 4) & 1) * 8, k_sel = (lane >> 3) & 1;
-  const int v_tok = (lane & 7) + ((lane >> 3) & 1) * 8, v_sel = (lane >> 4) & 1;
-  const uint32_t k_row = k_tok * 128, k_key = k_tok & 7;
-  const uint32_t v_row = v_tok * 128, v_key = v_tok & 7;
-
-  while (true) {
-    int item = 0;
-    if (lane == 0) item = atomicAdd(counter, 1);
-    item = __shfl_sync(0xffffffffu, item, 0);
-    if (item >= total_items) break;
-    const int sci = item / p.kv_heads, h = item % p.kv_heads;
-    const int b = p.sc.item_seq[sci], ck = p.sc.item_chunk[sci];
-    const long long rl = read_length(p.lengths, p.positions, b, capacity_tokens, nullptr);
-    const int nchunks = p.sc.offsets[b + 1] - p.sc.offsets[b];
-    const long long t_begin = (long long)ck * chunk;
-    const long long t_end = rl < t_begin + chunk ? rl : t_begin + chunk;
-    const int ntiles = (int)((t_end - t_begin + kTileTokens - 1) / kTileTokens);
-
-    // Query fragments: rows g < group are real heads, the rest of the 16 MMA rows are zero.
-    uint32_t qa[8][2];
-    {
-      const bool real = g < p.group;
-      const T* qrow = reinterpret_cast<const T*>(p.q.ptr) + (long long)b * p.q.s[0] +
-                      (long long)(h * p.group + (real ? g : 0)) * p.q.s[1];
-#pragma unroll
-      for (int ks = 0; ks < 8; ++ks) {
-        const uint32_t lo = *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 2 * t);
-        const uint32_t hi = *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 8 + 2 * t);
-        qa[ks][0] = real ? lo : 0u;
-        qa[ks][1] = real ? hi : 0u;
-      }
-    }
-
-    float m = -INFINITY, l = 0.f;
-    float o[16][4];
-#pragma unroll
-    for (int n = 0; n < 16; ++n) o[n][0] = o[n][1] = o[n][2] = o[n][3] = 0.f;
-
-    bool timed_out = false;
-    for (int batch0 = 0; batch0 < ntiles && !timed_out; batch0 += kPidBatch) {
-      const int nb = ntiles - batch0 < kPidBatch ? ntiles - batch0 : kPidBatch;
-      __syncwarp();
-      for (int i = lane; i < nb; i += 32) {
-        const long long tok = t_begin + (long long)(batch0 + i) * kTileTokens;
-        long long pid = p.tables.at(b, tok / p.block_size);
-        if (pid < 0 || pid >= p.num_blocks) {
-          raise_status(p.status, MIE_STATUS_BAD_PAGE);
-          pid = 0;
-        }
-        pids[i] = (int)pid;
-      }
-      __syncwarp();
-      auto issue = [&](int i) {
-        const int s = i % kStages;
-        const long long tok = t_begin + (long long)(batch0 + i) * kTileTokens;
-        const int tok_in_page = (int)(tok % p.block_size);
-        uint8_t* dst = stages + (size_t)s * kStageBytes;
-        mbar_expect_tx(&bars[s], kStageBytes);
-        tma_load_4d_hint(dst, &kmap, &bars[s], 0, tok_in_page, h, pids[i], stream_policy);
-        tma_load_4d_hint(dst + kTileBytes / 2, &kmap, &bars[s], 64, tok_in_page, h, pids[i], stream_policy);
-        tma_load_4d_hint(dst + kTileBytes, &vmap, &bars[s], 0, tok_in_page, h, pids[i], stream_policy);
-        tma_load_4d_hint(dst + kTileBytes + kTileBytes / 2, &vmap, &bars[s], 64, tok_in_page, h, pids[i],
-                         stream_policy);
-      };
-      if (lane == 0) {
-        for (int i = 0; i < kStages && i < nb; ++i) issue(i);
-      }
-      for (int i = 0; i < nb; ++i) {
-        const int s = i % kStages;
-        const bool arrived = mbar_wait_bounded(&bars[s], (parity >> s) & 1u);
-        if (!__all_sync(0xffffffffu, arrived)) {
-          timed_out = true;
-          break;
-        }
-        parity ^= 1u << s;
-        const uint32_t kbase = smem_u32(stages + (size_t)s * kStageBytes);
-        const uint32_t vbase = kbase + kTileBytes;
-        const long long tok0 = t_begin + (long long)(batch0 + i) * kTileTokens;
-        const int valid = (int)(t_end - tok0 < kTileTokens ? t_end - tok0 : kTileTokens);
-
-        if (valid < kTileTokens) {
-          // Rows past the read length may hold anything (even NaN bits): zero
-          // them in V so that 0 * V stays 0.  K rows are masked by select below.
-          uint8_t* vt = stages + (size_t)s * kStageBytes + kTileBytes;
-          for (int c = lane; c < 2 * kTileTokens * 8; c += 32) {
-            const int half = c / (kTileTokens * 8), rem = c % (kTileTokens * 8);
-            const int row = rem / 8;
-            if (row >= valid) {
-              *reinterpret_cast<uint4*>(vt + half * (kTileBytes / 2) + row * 128 + (rem % 8) * 16) =
-                  make_uint4(0, 0, 0, 0);
-            }
-          }
-          fence_proxy_async_smem();
-          __syncwarp();
-        }
-
-        // S = Q K^T for 16 tokens: two n-tiles, two accumulator sets to shorten the chain.
-        float sa[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-        float sb[2][4] = {{0.f, 0.f, 0.f, 0.f}, {0.f, 0.f, 0.f, 0.f}};
-#pragma unroll
-        for (int ks = 0; ks < 8; ++ks) {
-          const uint32_t addr =
-              kbase + (ks >> 2) * (kTileBytes / 2) + k_row + (((((ks & 3) * 2) | k_sel) ^ k_key) << 4);
-          uint32_t r0, r1, r2, r3;
-          ldmatrix_x4(r0, r1, r2, r3, addr);
-          if (ks & 1) {
-            Mma16816<T>::run(sb[0], qa[ks][0], 0u, qa[ks][1], 0u, r0, r1);
-            Mma16816<T>::run(sb[1], qa[ks][0], 0u, qa[ks][1], 0u, r2, r3);
-          } else {
-            Mma16816<T>::run(sa[0], qa[ks][0], 0u, qa[ks][1], 0u, r0, r1);
-            Mma16816<T>::run(sa[1], qa[ks][0], 0u, qa[ks][1], 0u, r2, r3);
-          }
-        }
-        // This lane's four scores of head g: tokens 2t, 2t+1, 8+2t, 9+2t.  The reference keeps the
-        // Q.K^T product in the activation dtype (a bf16/fp16 bmm per page) before the fp32 softmax;
-        // rounding the fp32 dot product once reproduces that.
-        float sv[4];
-        sv[0] = round_act<T>(sa[0][0] + sb[0][0]) * p.scale_log2;
-        sv[1] = round_act<T>(sa[0][1] + sb[0][1]) * p.scale_log2;
-        sv[2] = round_act<T>(sa[1][0] + sb[1][0]) * p.scale_log2;
-        sv[3] = round_act<T>(sa[1][1] + sb[1][1]) * p.scale_log2;
-        const int tk = 2 * t;
-        if (tk >= valid) sv[0] = -INFINITY;
-        if (tk + 1 >= valid) sv[1] = -INFINITY;
-        if (tk + 8 >= valid) sv[2] = -INFINITY;
-        if (tk + 9 >= valid) sv[3] = -INFINITY;
-        float mx = fmaxf(fmaxf(sv[0], sv[1]), fmaxf(sv[2], sv[3]));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 1));
-        mx = fmaxf(mx, __shfl_xor_sync(0xffffffffu, mx, 2));
-        const float m_new = fmaxf(m, mx);  // finite: token 0 of a tile is always valid
-        const float alpha = exp2f(m - m_new);
-        const float p0 = exp2f(sv[0] - m_new), p1 = exp2f(sv[1] - m_new);
-        const float p2 = exp2f(sv[2] - m_new), p3 = exp2f(sv[3] - m_new);
-        l = l * alpha + ((p0 + p1) + (p2 + p3));
-        m = m_new;
-        // P.V runs on the tensor cores in the activation dtype; the reference multiplies fp32 weights by
-        // fp32 V, so P is split into a rounded part and its remainder (two MMAs) to keep ~16 more bits.
-        const uint32_t pa0 = Mma16816<T>::pack(p0, p1), pa2 = Mma16816<T>::pack(p2, p3);
-        const uint32_t pb0 = Mma16816<T>::pack(p0 - round_act<T>(p0), p1 - round_act<T>(p1));
-        const uint32_t pb2 = Mma16816<T>::pack(p2 - round_act<T>(p2), p3 - round_act<T>(p3));
-#pragma unroll
-        for (int n = 0; n < 16; ++n) {
-          o[n][0] *= alpha;
-          o[n][1] *= alpha;
-        }
-        // O += P V
-#pragma unroll
-        for (int np = 0; np < 8; ++np) {
-          const uint32_t addr =
-              vbase + (np >> 2) * (kTileBytes / 2) + v_row + (((((np & 3) * 2) | v_sel) ^ v_key) << 4);
-          uint32_t r0, r1, r2, r3;
-          ldmatrix_x4_trans(r0, r1, r2, r3, addr);
-          Mma16816<T>::run(o[2 * np], pa0, 0u, pa2, 0u, r0, r1);
-          Mma16816<T>::run(o[2 * np + 1], pa0, 0u, pa2, 0u, r2, r3);
-          Mma16816<T>::run(o[2 * np], pb0, 0u, pb2, 0u, r0, r1);
-          Mma16816<T>::run(o[2 * np + 1], pb0, 0u, pb2, 0u, r2, r3);
-        }
-        __syncwarp();
-        if (lane == 0 && i + kStages < nb) issue(i + kStages);
-      }
-    }
-    if (timed_out) {
-      if (lane == 0) raise_status(p.status, MIE_STATUS_WAIT_TIMEOUT);
-      break;
-    }
-
-    // Row sum over the quad, then write the result (final or partial).
-    l += __shfl_xor_sync(0xffffffffu, l, 1);
-    l += __shfl_xor_sync(0xffffffffu, l, 2);
-    const bool head_live = g < p.group;
-    const int head = h * p.group + (head_live ? g : 0);
-    if (nchunks == 1) {
-      const float inv = 1.f / fmaxf(l, 1.17549435e-38f);
-      T* orow = reinterpret_cast<T*>(p.out.ptr) + (long long)b * p.out.s[0] + (long long)head * p.out.s[1];
-      float amax = 0.f;
-#pragma unroll
-      for (int n = 0; n < 16; ++n) {
-        o[n][0] = round_act<T>(o[n][0] * inv);  // the stored (and quantised) value is the rounded one
-        o[n][1] = round_act<T>(o[n][1] * inv);
-        amax = fmaxf(amax, fmaxf(fabsf(o[n][0]), fabsf(o[n][1])));
-        if (head_live) *reinterpret_cast<uint32_t*>(orow + n * 8 + 2 * t) = Mma16816<T>::pack(o[n][0], o[n][1]);
-      }
-      if (p.out_q8 != nullptr) {
-        amax = fmaxf(amax, __shfl_xor_sync(0xffffffffu, amax, 1));
-        amax = fmaxf(amax, __shfl_xor_sync(0xffffffffu, amax, 2));
-        const float scale = __fdiv_rn(amax, 448.0f), denom = fmaxf(scale, 1e-12f);
-        if (head_live) {
-          uint8_t* qrow = p.out_q8 + (long long)b * p.ldq8 + head * kHeadDim;
-#pragma unroll
-          for (int n = 0; n < 16; ++n) {
-            *reinterpret_cast<__nv_fp8x2_storage_t*>(qrow + n * 8 + 2 * t) = __nv_cvt_float2_to_fp8x2(
-                make_float2(__fdiv_rn(o[n][0], denom), __fdiv_rn(o[n][1], denom)), __NV_SATFINITE, __NV_E4M3);
-          }
-          if (t == 0) p.out_scales[(long long)head * p.out_scale_ld + b] = scale;
-        }
-      }
-    } else {
-      const long long first_row = (long long)p.sc.offsets[b] * p.q_heads;
-      if (head_live) {
-        const long long row = first_row + (long long)ck * p.q_heads + head;
-        float* po = p.sc.part_o + row * kHeadDim;
-#pragma unroll
-        for (int n = 0; n < 16; ++n) {
-          *reinterpret_cast<float2*>(po + n * 8 + 2 * t) = make_float2(o[n][0], o[n][1]);
-        }
-        if (t == 0) {
-          p.sc.part_m[row] = m;
-          p.sc.part_l[row] = l;
-        }
-      }
-    }
-  }
-
-  // Requests with nothing to read (rejected metadata) get zeros.
-  const int warps_total = gridDim.x * kWarps;
-  for (int e = blockIdx.x * kWarps + warp; e < p.batch; e += warps_total) {
-    if (p.sc.offsets[e + 1] != p.sc.offsets[e]) continue;
-    for (int hq = 0; hq < p.q_heads; ++hq) {
-      T* orow = reinterpret_cast<T*>(p.out.ptr) + (long long)e * p.out.s[0] + (long long)hq * p.out.s[1];
-      *reinterpret_cast<uint2*>(orow + 4 * lane) = make_uint2(0u, 0u);
-      if (p.out_q8 != nullptr) {
-        *reinterpret_cast<uint32_t*>(p.out_q8 + (long long)e * p.ldq8 + hq * kHeadDim + 4 * lane) = 0u;
-        if (lane == 0) p.out_scales[(long long)hq * p.out_scale_ld + e] = 0.f;
-      }
-    }
-  }
-}
 
 // ---------------------------------------------------------------------------
 // Main kernel over an e4m3 K/V pool (one fp32 scale per token and KV head)
@@ -1022,10 +518,10 @@ __global__ void generic_decode_kernel(View4 q, View4 out, View4 kb, View4 vb, In
 struct MapKey {
   void* ptr;
   long long s0, s1, s2;
-  int num_blocks, kv_heads, block_size, dtype;
+  int num_blocks, kv_heads, block_size, dim, dtype;
   bool operator==(const MapKey& o) const {
     return ptr == o.ptr && s0 == o.s0 && s1 == o.s1 && s2 == o.s2 && num_blocks == o.num_blocks &&
-           kv_heads == o.kv_heads && block_size == o.block_size && dtype == o.dtype;
+           kv_heads == o.kv_heads && block_size == o.block_size && dim == o.dim && dtype == o.dtype;
   }
 };
 struct MapKeyHash {
@@ -1034,16 +530,16 @@ struct MapKeyHash {
     h = h * 1000003u ^ (size_t)k.s0;
     h = h * 1000003u ^ (size_t)k.s1;
     h = h * 1000003u ^ (size_t)k.s2;
-    h = h * 1000003u ^ (size_t)(k.num_blocks * 131 + k.kv_heads * 17 + k.block_size * 3 + k.dtype);
+    h = h * 1000003u ^ (size_t)(k.num_blocks * 131 + k.kv_heads * 17 + k.block_size * 3 + k.dim * 7 + k.dtype);
     return h;
   }
 };
 
-int page_tensor_map(const mie_view4_t& pages, int num_blocks, int kv_heads, int block_size, int dtype,
+int page_tensor_map(const mie_view4_t& pages, int num_blocks, int kv_heads, int block_size, int dim, int dtype,
                     CUtensorMap* out) {
   static std::mutex mu;
   static std::unordered_map<MapKey, CUtensorMap, MapKeyHash> cache;
-  MapKey key{pages.ptr, pages.stride[0], pages.stride[1], pages.stride[2], num_blocks, kv_heads, block_size, dtype};
+  MapKey key{pages.ptr, pages.stride[0], pages.stride[1], pages.stride[2], num_blocks, kv_heads, block_size, dim, dtype};
   {
     std::lock_guard<std::mutex> lock(mu);
     auto it = cache.find(key);
@@ -1052,7 +548,7 @@ int page_tensor_map(const mie_view4_t& pages, int num_blocks, int kv_heads, int 
       return MIE_OK;
     }
   }
-  const uint64_t dims[4] = {(uint64_t)kHeadDim, (uint64_t)block_size, (uint64_t)kv_heads, (uint64_t)num_blocks};
+  const uint64_t dims[4] = {(uint64_t)dim, (uint64_t)block_size, (uint64_t)kv_heads, (uint64_t)num_blocks};
   const uint64_t strides[3] = {(uint64_t)pages.stride[2] * 2, (uint64_t)pages.stride[1] * 2,
                                (uint64_t)pages.stride[0] * 2};
   const uint32_t box[4] = {64, kTileTokens, 1, 1};
@@ -1077,50 +573,7 @@ bool pages_fit_tma(const mie_view4_t& v, int head_dim, int block_size) {
 
 namespace {
 
-constexpr size_t kDecodeSmem = (size_t)kWarps * kStages * kStageBytes + kWarps * kStages * 8 +
-                               (size_t)kWarps * kPidBatch * 4 + 1024;
-
-long long fixed_scratch_bytes(int batch, int kv_heads) {
-  (void)kv_heads;
-  return kHeaderInts * 4 + align_up((long long)(batch + 1) * 4, 256);
-}
-long long per_chunk_bytes(int q_heads, int head_dim) { return 8 + (long long)q_heads * (head_dim + 2) * 4; }
-
-// (request, chunk) pairs `mie_decode_scratch_bytes` makes room for beyond one per request: four items per
-// warp.  The plan kernel considers more items per warp only while they fit the scratch it was given.
-// One thread per request, at least two warps, at most the kernel's bound: a small batch does not pay for
-// block-wide reductions over 32 warps.
-int plan_threads(int batch) {
-  const int threads = (batch + 31) / 32 * 32;
-  return threads < 64 ? 64 : threads > kPlanThreads ? kPlanThreads : threads;
-}
-
-int target_seq_chunks(int kv_heads) {
-  const int items = sm_count() * kWarps * 4;
-  return (items + kv_heads - 1) / kv_heads;
-}
-
-Scratch carve(void* scratch, long long bytes, int batch, int q_heads, int kv_heads, int head_dim) {
-  Scratch s;
-  char* base = reinterpret_cast<char*>(scratch);
-  s.header = reinterpret_cast<int*>(base);
-  s.offsets = reinterpret_cast<int*>(base + kHeaderInts * 4);
-  long long off = fixed_scratch_bytes(batch, kv_heads);
-  const long long avail = bytes - off - 1024;
-  long long cap = avail / per_chunk_bytes(q_heads, head_dim);
-  if (cap > 0x3fffffff) cap = 0x3fffffff;
-  s.cap = (int)(cap > 0 ? cap : 0);
-  s.item_seq = reinterpret_cast<int*>(base + off);
-  off += align_up((long long)s.cap * 4, 256);
-  s.item_chunk = reinterpret_cast<int*>(base + off);
-  off += align_up((long long)s.cap * 4, 256);
-  s.part_m = reinterpret_cast<float*>(base + off);
-  off += align_up((long long)s.cap * q_heads * 4, 256);
-  s.part_l = reinterpret_cast<float*>(base + off);
-  off += align_up((long long)s.cap * q_heads * 4, 256);
-  s.part_o = reinterpret_cast<float*>(base + off);
-  return s;
-}
+constexpr size_t kDecodeSmem = DecodeTile<2, 2>::kSmem;
 
 // Warps per query head in the merge: the chunks of a request are shared by W warps, so the longest request
 // (tens of chunks) sets the length of the kernel.  With many blocks (request x KV head) two warps per head
@@ -1147,10 +600,10 @@ int launch_fast(const DecodeParams& p, const CUtensorMap& kmap, const CUtensorMa
   int dev = 0;
   MIE_CUDA(cudaGetDevice(&dev));
   if (dev >= 0 && dev < 64 && !configured[dev]) {
-    MIE_CUDA(cudaFuncSetAttribute(decode_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kDecodeSmem));
+    MIE_CUDA(cudaFuncSetAttribute(decode_kernel<T, 2, 2, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, (int)kDecodeSmem));
     configured[dev] = true;
   }
-  MIE_CUDA(launch_chained(decode_kernel<T>, dim3(sm_count()), dim3(kWarps * 32), kDecodeSmem, stream, kmap, vmap, p));
+  MIE_CUDA(launch_chained(decode_kernel<T, 2, 2, false>, dim3(sm_count()), dim3(kWarps * 32), kDecodeSmem, stream, kmap, vmap, p));
   MIE_LAUNCH_CHECK("decode_kernel");
   // Groups wider than kMaxGroupMerge take several passes of head sub-groups.
   for (int g0 = 0; g0 < p.group; g0 += kMaxGroupMerge) {
@@ -1249,17 +702,17 @@ extern "C" int mie_paged_decode_attention(mie_view4_t query, mie_view4_t out, mi
   DecodeParams p{View4(query), View4(out), IndexView(block_tables), IndexView(sequence_lengths),
                  IndexView(query_positions), sc, batch, q_heads, kv_heads, group, block_size, num_blocks,
                  table_width, scale * 1.4426950408889634f, plan_slot, status, reinterpret_cast<uint8_t*>(out_q8), ldq8,
-                 out_scales, out_scale_ld, 0};
+                 out_scales, out_scale_ld, 0, head_dim, head_dim, kv_heads, 0, nullptr};
   if (!use_plan) {
     plan_kernel<<<1, plan_threads(batch), 0, stream>>>(p.lengths, p.positions, batch, (long long)table_width * block_size,
-                                                kv_heads, split_policy, sm_count() * kWarps, 128, sc, status);
+                                                kv_heads, split_policy, sm_count() * kWarps, 128, 0ll, sc, status);
     MIE_LAUNCH_CHECK("plan_kernel");
   }
   if (plan_only) return MIE_OK;
 
   CUtensorMap kmap, vmap;
-  if (int rc = page_tensor_map(key_blocks, num_blocks, kv_heads, block_size, dtype, &kmap)) return rc;
-  if (int rc = page_tensor_map(value_blocks, num_blocks, kv_heads, block_size, dtype, &vmap)) return rc;
+  if (int rc = page_tensor_map(key_blocks, num_blocks, kv_heads, block_size, head_dim, dtype, &kmap)) return rc;
+  if (int rc = page_tensor_map(value_blocks, num_blocks, kv_heads, block_size, head_dim, dtype, &vmap)) return rc;
   if (dtype == MIE_DTYPE_BF16) return launch_fast<__nv_bfloat16>(p, kmap, vmap, stream);
   return launch_fast<__half>(p, kmap, vmap, stream);
 }
@@ -1380,10 +833,10 @@ extern "C" int mie_paged_decode_attention_kv8(mie_view4_t query, mie_view4_t out
   DecodeParams p{View4(query), View4(out), IndexView(block_tables), IndexView(sequence_lengths),
                  IndexView(query_positions), sc, batch, q_heads, kv_heads, q_heads / kv_heads, kTileTokens, num_blocks,
                  table_width, scale * 1.4426950408889634f, plan_slot, status, reinterpret_cast<uint8_t*>(out_q8), ldq8,
-                 out_scales, out_scale_ld, 0};
+                 out_scales, out_scale_ld, 0, kHeadDim, kHeadDim, kv_heads, 0, nullptr};
   if (!use_plan) {
     plan_kernel<<<1, plan_threads(batch), 0, stream>>>(p.lengths, p.positions, batch, (long long)table_width * kTileTokens,
-                                                kv_heads, split_policy, sm_count() * kWarps8, 256, sc, status);
+                                                kv_heads, split_policy, sm_count() * kWarps8, 256, 0ll, sc, status);
     MIE_LAUNCH_CHECK("plan_kernel");
   }
   if (plan_only) return MIE_OK;

@@ -18,7 +18,7 @@
 namespace mie {
 
 // Defined in decode_attention.cu: cached 4-D tensor map over [pages, kv_heads, page, 128].
-int page_tensor_map(const mie_view4_t& pages, int num_blocks, int kv_heads, int block_size, int dtype,
+int page_tensor_map(const mie_view4_t& pages, int num_blocks, int kv_heads, int block_size, int dim, int dtype,
                     CUtensorMap* out);
 bool pages_fit_tma(const mie_view4_t& v, int head_dim, int block_size);
 // Defined in prefill_attention_umma.cu: the tcgen05 kernel; MIE_ERR_UNSUPPORTED when the shape does not fit it.
@@ -332,8 +332,8 @@ extern "C" int mie_flash_prefill_attention(const void* query, int64_t q_token_st
     if (rc != MIE_ERR_UNSUPPORTED) return rc;
   }
   CUtensorMap kmap, vmap;
-  if (int rc = page_tensor_map(key_blocks, num_blocks, kv_heads, block_size, dtype, &kmap)) return rc;
-  if (int rc = page_tensor_map(value_blocks, num_blocks, kv_heads, block_size, dtype, &vmap)) return rc;
+  if (int rc = page_tensor_map(key_blocks, num_blocks, kv_heads, block_size, head_dim, dtype, &kmap)) return rc;
+  if (int rc = page_tensor_map(value_blocks, num_blocks, kv_heads, block_size, head_dim, dtype, &vmap)) return rc;
   PrefillParams p{(const char*)query, q_token_stride, q_head_stride, (char*)out, o_token_stride, o_head_stride,
                   IndexView(block_tables), IndexView(cu_seqlens), IndexView(kv_lens), requests, q_heads, kv_heads,
                   group, block_size, num_blocks, table_width, scale * 1.4426950408889634f, status};

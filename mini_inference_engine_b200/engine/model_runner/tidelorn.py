@@ -25,13 +25,21 @@ from dataclasses import dataclass
 import torch
 
 from ..kernels.decoder_glue import clamped_glu, embed_tokens, qkv_norm_mix_write, sum_rms_norm
-from ..kv_cache.sink_attention import attention_rows
+from ..kv_cache.sink_attention import (
+    attention_rows,
+    sink_decode_attention,
+    sink_decode_supported,
+    sink_prefill_attention,
+    sink_prefill_supported,
+)
+from ..kv_cache.triton_paged_attention import decode_scratch
 from ... import _lib
 from .step_runner import PagedStepRunner
 
 SINUSOID_BASE = 10000.0
 GATE_SLOPE = 1.702
 UP_OFFSET = 1.0
+PLAN_SLOTS = 64  # work counters of one decode work plan
 NORM_WEIGHT_OFFSET = 1.0  # norm weights are stored as their deviation from one
 
 
@@ -221,7 +229,12 @@ class TidelornRunner(PagedStepRunner):
 
     def __init__(self, weights: TidelornWeights, *, num_pages: int, max_batch: int, max_context: int,
                  decode_buckets: tuple[int, ...] | None = None, chunk_buckets: tuple[int, ...] = (128, 512),
-                 max_chunks: int = 4, kv_init: str = "zeros") -> None:
+                 max_chunks: int = 4, kv_init: str = "zeros", attention: str = "auto") -> None:
+        """``attention``: "auto" takes the streaming kernels where a layer's sizes and number format allow them,
+        "rows" the row kernel everywhere."""
+
+        if attention not in ("auto", "rows"):
+            raise ValueError("attention must be 'auto' or 'rows'")
         super().__init__(weights.shape, weights.device, num_pages=num_pages, max_batch=max_batch,
                          max_context=max_context, decode_buckets=decode_buckets, chunk_buckets=chunk_buckets,
                          max_chunks=max_chunks)
@@ -237,6 +250,21 @@ class TidelornRunner(PagedStepRunner):
                 if kv_init == "normal":
                     blocks.normal_()
                 pool.append(blocks)
+        # Layers of one geometry share a split-KV work plan within a step, and its scratch: (scratch key, streams
+        # decode rows, streams chunks) per layer.
+        self._attention: list[tuple[tuple, bool, bool]] = []
+        self._scratch: dict[tuple, torch.Tensor] = {}
+        rows = max(max_batch, self.decode_buckets[-1])
+        for layer in self.shape.layers:
+            sizes = (layer.dim, layer.vdim, self.shape.page, self.dtype)
+            decode = attention == "auto" and sink_decode_supported(*sizes)
+            chunks = attention == "auto" and sink_prefill_supported(layer.heads, layer.kv_heads, *sizes, layer.scale)
+            key = (layer.heads, layer.kv_heads, layer.dim, layer.vdim, layer.window)
+            if decode and key not in self._scratch:
+                reach = max_context if layer.window is None else min(max_context, layer.window + 16)
+                self._scratch[key] = decode_scratch(rows, layer.heads, layer.kv_heads, layer.vdim, rows * reach,
+                                                    self.device)
+            self._attention.append((key, decode, chunks))
         self.history = torch.zeros(self.total_pages, self.shape.page, dtype=torch.int32, device=self.device)
 
     # -- projections ----------------------------------------------------------------------------
@@ -265,11 +293,34 @@ class TidelornRunner(PagedStepRunner):
     # -- the layers -----------------------------------------------------------------------------
 
     def _attend(self, index: int, queries: torch.Tensor, attended: torch.Tensor, positions, token_to_sequence,
-                block_tables, **_) -> None:
-        layer, weights = self.shape.layers[index], self.weights.layers[index]
-        attention_rows(queries, attended, self.key_blocks[index], self.value_blocks[index], positions,
-                       token_to_sequence, block_tables, scale=layer.scale, window=layer.window, sinks=weights.sinks,
-                       status=self.status)
+                block_tables, plans: dict, *, decode_rows: int, decode_lengths, cu_seqlens=None, kv_lens=None,
+                max_query_len: int = 0) -> None:
+        """Attention of one layer: the leading ``decode_rows`` rows, then the packed chunks.  ``plans`` counts the
+        layers that have used each work plan of this step."""
+
+        layer, sinks = self.shape.layers[index], self.weights.layers[index].sinks
+        keys, values = self.key_blocks[index], self.value_blocks[index]
+        common = dict(scale=layer.scale, window=layer.window, sinks=sinks, status=self.status)
+        key, stream_decode, stream_chunks = self._attention[index]
+        parts = []  # row ranges left to the row kernel
+        if decode_rows and stream_decode:
+            used = plans.get(key, 0)
+            plans[key] = used + 1
+            sink_decode_attention(queries[:decode_rows], attended[:decode_rows], keys, values,
+                                  block_tables[:decode_rows], decode_lengths, scratch=self._scratch[key],
+                                  use_plan=used % PLAN_SLOTS != 0, plan_slot=used % PLAN_SLOTS, **common)
+        elif decode_rows:
+            parts.append(slice(0, decode_rows))
+        if queries.shape[0] > decode_rows:
+            if stream_chunks:
+                sink_prefill_attention(queries[decode_rows:], attended[decode_rows:], keys, values,
+                                       block_tables[decode_rows:], cu_seqlens, kv_lens, max_query_len=max_query_len,
+                                       **common)
+            else:
+                parts.append(slice(decode_rows, queries.shape[0]))
+        for rows in parts:
+            attention_rows(queries[rows], attended[rows], keys, values, positions[rows],
+                           None if token_to_sequence is None else token_to_sequence[rows], block_tables, **common)
 
     def _layers(self, input_ids, positions, token_to_sequence, block_tables, **batch) -> torch.Tensor:
         """Residual rows after the last layer (fp32), the cache holding the new tokens."""
@@ -280,7 +331,7 @@ class TidelornRunner(PagedStepRunner):
                               scale=shape.embed_scale, page=shape.page, num_pages=self.total_pages,
                               bigram=weights.bigram, mul_prev=shape.mul_prev, mul_cur=shape.mul_cur,
                               history=self.history, frequencies=weights.frequencies, status=self.status)
-        v_first = None
+        v_first, plans = None, {}
         norm = dict(eps=shape.eps, alpha=shape.alpha, weight_offset=NORM_WEIGHT_OFFSET)
         for index, (layer, w) in enumerate(zip(shape.layers, weights.layers)):
             qkv = self._linear(x, w.qkv, w.qkv_bias)
@@ -293,7 +344,7 @@ class TidelornRunner(PagedStepRunner):
             if index == shape.first_v_mix:
                 v_first = qkv[:, (layer.heads + layer.kv_heads) * layer.dim:]
             attended = torch.empty(tokens, layer.heads, layer.vdim, dtype=self.dtype, device=self.device)
-            self._attend(index, queries, attended, positions, token_to_sequence, block_tables, **batch)
+            self._attend(index, queries, attended, positions, token_to_sequence, block_tables, plans, **batch)
             mixed = self._linear(attended.view(tokens, layer.heads * layer.vdim), w.o)
             x32, x = sum_rms_norm(x32, mixed, w.norm1, **norm)
             if layer.ff is not None:
