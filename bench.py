@@ -47,8 +47,9 @@ def parse_args() -> argparse.Namespace:
     parser.add_argument("--layers", type=int, default=None, help="debug: fewer layers (invalid as a result)")
     parser.add_argument("--no-cpu-baseline", action="store_true")
     parser.add_argument("--no-e2e", action="store_true")
-    parser.add_argument("--workload", default="config4", choices=["config4", "config3"],
-                        help="config4: ragged decode sweep point (the headline); config3: 8 x (2048 prompt + 128 new)")
+    parser.add_argument("--workload", default="config4", choices=["config4", "config3", "tidelorn"],
+                        help="config4: ragged decode sweep point (the headline); config3: 8 x (2048 prompt + 128 new); "
+                             "tidelorn: that design's prefill, decode and kernels beside the Qwen3 runner")
     parser.add_argument("--no-extras", action="store_true",
                         help="skip the extra keys measured after the headline (configs 0-3, FP8 KV cache)")
     parser.add_argument("--breakdown", action="store_true",
@@ -66,6 +67,17 @@ def measured_peaks() -> tuple[float, str]:
         except (ValueError, KeyError):
             pass
     return FALLBACK_HBM_GBS, "fallback"
+
+
+FALLBACK_BF16_TFLOPS = 1590.0
+
+
+def measured_tensor_peak() -> float:
+    path = ROOT / "MEASURED_PEAKS.json"
+    try:
+        return float(json.loads(path.read_text())["bf16_tflops"])
+    except (OSError, ValueError, KeyError):
+        return FALLBACK_BF16_TFLOPS
 
 
 # ----------------------------------------------------------------------------------------------
@@ -286,6 +298,21 @@ def run_config3(args, shape, device, rank, world, group) -> None:
         })
     if world > 1:
         leave_together(runner, device)
+
+
+def run_tidelorn(args, device, rank) -> None:
+    """Not the headline: prefill and decode of the Tidelorn design at layer sizes of real models, beside the
+    Qwen3 runner at equal sizes, with every kernel of both against its roofline."""
+
+    import modelbench
+
+    sampler = ClockSampler(device.index or 0)
+    sampler.start()
+    result = modelbench.run(device, measured_peaks()[0], measured_tensor_peak())
+    clocks = sampler.stop()
+    if rank == 0:
+        emit({"workload": "tidelorn", "n_gpus": 1, "data": "synthetic", "dtype": "bf16 (Qwen3 arm: fp8_e4m3 GEMM)",
+              "peaks": measured_peaks()[1], "clocks": clocks, **result})
 
 
 def run_breakdown(runner, buffers, steps: int, device, rank: int, world: int, concurrency: int) -> None:
@@ -537,6 +564,9 @@ def main() -> None:
         return float(t.item())
 
     shape = Qwen3Shape()
+    if args.workload == "tidelorn":
+        run_tidelorn(args, device, rank)
+        return
     if args.workload == "config3":
         run_config3(args, shape, device, rank, world, group)
         return

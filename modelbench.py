@@ -1,0 +1,253 @@
+"""Prefill and decode throughput of a model design at layer sizes of real models, beside the Qwen3 runner at equal
+sizes, and every kernel of both against its roofline (``bench.py --workload tidelorn``).
+
+Random weights.  ``Tidelorn`` here alternates whole-prefix and 1,024-token-window layers.  Decode is a replayed CUDA
+graph of one step at a uniform context; prefill is one packed forward of whole prompts.  Kernels are timed alone with
+CUDA events, L2 flushed before each (median of the repeats): a kernel's fraction is (bytes / time / copy peak) or
+(FLOPs / time / tensor peak).
+"""
+
+from __future__ import annotations
+
+import gc
+import statistics
+
+import torch
+
+from mini_inference_engine_b200.engine.kernels.decoder_glue import (
+    clamped_glu,
+    embed_tokens,
+    qkv_norm_mix_write,
+    sum_rms_norm,
+)
+from mini_inference_engine_b200.engine.kv_cache.sink_attention import sink_decode_attention, sink_prefill_attention
+from mini_inference_engine_b200.engine.kv_cache.triton_flash_prefill import launch_flash_prefill
+from mini_inference_engine_b200.engine.kv_cache.triton_paged_attention import launch_decode_attention
+from mini_inference_engine_b200.engine.model_runner.qwen3_decode import Qwen3DecodeRunner, Qwen3Shape, Qwen3Weights
+from mini_inference_engine_b200.engine.model_runner.tidelorn import TidelornRunner, TidelornShape, TidelornWeights
+
+# name: width, query heads, key/value heads, head size, feed-forward, vocabulary
+SIZES = {
+    "1.7b-layers": (2048, 16, 8, 128, 6144, 151936),
+    "4b-layers": (2560, 32, 8, 128, 9728, 151936),
+    "8b-layers": (4096, 32, 8, 128, 12288, 151936),
+}
+LAYERS = 8
+WINDOW = 1024
+
+
+def tidelorn_config(width, heads, kv_heads, dim, ff, vocab, layers=LAYERS, window=WINDOW) -> dict:
+    entries = []
+    for index in range(layers):
+        mixer = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5, "v_mix": True}
+        if index % 2 == 0:
+            mixer["q_temp"] = {"coef": 0.1, "every": 4096}
+        else:
+            mixer["mask"] = {"size": window}
+        entries.append({"type": "attention" if index % 2 == 0 else "attention_2", "mixer": mixer,
+                        "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}})
+    return {"vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 2.0, "layers": entries,
+            "embedding": {"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}}
+
+
+def _tables(batch: int, pages_each: int, total: int, device) -> torch.Tensor:
+    order = torch.randperm(total, generator=torch.Generator().manual_seed(1))[:batch * pages_each]
+    return order.to(torch.int32).view(batch, pages_each).to(device)
+
+
+def _event_ms(run, repeats: int, device) -> float:
+    start, end = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+    start.record()
+    for _ in range(repeats):
+        run()
+    end.record()
+    torch.cuda.synchronize(device)
+    return start.elapsed_time(end) / repeats
+
+
+class Flusher:
+    def __init__(self, device) -> None:
+        self.device, self.buffer = device, torch.empty(256 << 20, dtype=torch.uint8, device=device)
+
+    def median_us(self, run, repeats: int = 9) -> float:
+        for _ in range(3):
+            run()
+        samples = []
+        for _ in range(repeats):
+            self.buffer.zero_()
+            samples.append(_event_ms(run, 1, self.device) * 1e3)
+        return statistics.median(samples)
+
+
+def _throughput(runner, vocab: int, batch: int, context: int, prompts: int, prompt_len: int, steps: int, device) -> dict:
+    page = runner.shape.page
+    pages_each = -(-(context + steps + 16) // page)
+    buffers = runner.capture(batch, pages_each, advance=True)
+    buffers.block_tables.copy_(_tables(batch, pages_each, runner.num_pages, device))
+    buffers.input_ids.copy_(torch.randint(0, vocab, (batch,), device=device))
+    buffers.sequence_lengths.fill_(context + 1)
+    for _ in range(3):
+        runner.replay(batch, advance=True)
+    torch.cuda.synchronize(device)
+    decode_ms = _event_ms(lambda: runner.replay(batch, advance=True), steps, device)
+    tokens = prompts * prompt_len
+    ids = torch.randint(0, vocab, (tokens,), device=device)
+    owners = torch.arange(prompts, dtype=torch.int32, device=device).repeat_interleave(prompt_len)
+    positions = torch.arange(prompt_len, dtype=torch.int32, device=device).repeat(prompts)
+    tables = _tables(prompts, -(-prompt_len // page), runner.num_pages, device)
+    cu = torch.arange(prompts + 1, dtype=torch.int32, device=device) * prompt_len
+    lens = torch.full((prompts,), prompt_len, dtype=torch.int32, device=device)
+
+    def prefill():
+        runner.prefill_forward(ids, owners, positions, tables, cu, lens, prompt_len)
+
+    for _ in range(3):
+        prefill()
+    torch.cuda.synchronize(device)
+    prefill_ms = _event_ms(prefill, 5, device)
+    runner.check_status()
+    return {"decode": {"ms_per_step": decode_ms, "tok_per_s": batch / decode_ms * 1e3,
+                       "launches_of_this_library": runner.launches_per_step},
+            "prefill": {"ms": prefill_ms, "tok_per_s": tokens / prefill_ms * 1e3}}
+
+
+def _row(us: float, *, bytes_: float = 0.0, flops: float = 0.0, hbm: float, tensor: float) -> dict:
+    """Time beside the roofline time max(bytes / copy peak, FLOPs / tensor peak) of the same work."""
+
+    floor = max(bytes_ / (hbm * 1e9), flops / (tensor * 1e12)) * 1e6
+    return {"us": round(us, 2), "roofline_us": round(floor, 2), "frac": round(floor / us, 3)}
+
+
+def _kernels(size, tide: TidelornRunner, qwen: Qwen3DecodeRunner, batch, context, prompts, prompt_len, hbm, tensor,
+             device) -> dict:
+    width, heads, kv, dim, ff, vocab = size
+    flush, page = Flusher(device), tide.shape.page
+    w, q = tide.weights.layers[0], qwen.weights.layers[0]
+    layer = tide.shape.layers[0]
+    out = {}
+
+    def pair(name, ours, theirs, *, work, their_work=None):
+        their_work = their_work or work
+        a = _row(flush.median_us(ours), hbm=hbm, tensor=tensor, **work)
+        b = _row(flush.median_us(theirs), hbm=hbm, tensor=their_work.pop("tensor", tensor), **their_work)
+        out[name] = {"tidelorn": a, "qwen3": b, "distance_ratio": round(b["frac"] / a["frac"], 2)}
+
+    def bf16(*shape):
+        return torch.randn(*shape, device=device).to(torch.bfloat16)
+
+    # Decode attention over a uniform context, and the windowed form of it.
+    tables = _tables(batch, -(-context // page), tide.num_pages, device)
+    lengths = torch.full((batch,), context, dtype=torch.int32, device=device)
+    queries, attended = bf16(batch, heads, dim), bf16(batch, heads, dim)
+    kv_bytes = 2 * kv * dim * 2
+
+    def tide_decode(window):
+        key = next(k for k, layer in zip((a[0] for a in tide._attention), tide.shape.layers) if layer.window == window)
+        return lambda: sink_decode_attention(queries, attended, tide.key_blocks[0], tide.value_blocks[0], tables,
+                                             lengths, scale=layer.scale, window=window, sinks=w.sinks,
+                                             scratch=tide._scratch[key], status=tide.status)
+
+    def qwen_decode():
+        launch_decode_attention(queries.unsqueeze(2), attended.unsqueeze(2), qwen.key_blocks[0], qwen.value_blocks[0],
+                                tables, lengths, None, scale=layer.scale, max_total_tokens=batch * context,
+                                scratch=qwen.scratch, split_policy=1, status=qwen.status)
+
+    pair("decode attention", tide_decode(None), qwen_decode, work={"bytes_": batch * context * kv_bytes})
+    reach = min(context, WINDOW)
+    pair("decode attention, window", tide_decode(WINDOW), qwen_decode, work={"bytes_": batch * reach * kv_bytes},
+         their_work={"bytes_": batch * context * kv_bytes})
+
+    # Prefill attention of whole prompts.
+    tokens = prompts * prompt_len
+    queries_p, attended_p = bf16(tokens, heads, dim), bf16(tokens, heads, dim)
+    tables_p = _tables(prompts, -(-prompt_len // page), tide.num_pages, device)
+    cu = torch.arange(prompts + 1, dtype=torch.int32, device=device) * prompt_len
+    lens = torch.full((prompts,), prompt_len, dtype=torch.int32, device=device)
+
+    def tide_prefill(window):
+        return lambda: sink_prefill_attention(queries_p, attended_p, tide.key_blocks[0], tide.value_blocks[0], tables_p,
+                                              cu, lens, max_query_len=prompt_len, scale=layer.scale, window=window,
+                                              sinks=w.sinks, status=tide.status)
+
+    def qwen_prefill():
+        launch_flash_prefill(queries_p, attended_p, qwen.key_blocks[0], qwen.value_blocks[0], tables_p, cu, lens,
+                             max_query_len=prompt_len, scale=layer.scale, status=qwen.status)
+
+    seen = prompts * prompt_len * (prompt_len + 1) / 2
+    inside = prompts * (WINDOW * prompt_len - WINDOW * (WINDOW - 1) / 2 if prompt_len > WINDOW
+                        else prompt_len * (prompt_len + 1) / 2)
+    pair("prefill attention", tide_prefill(None), qwen_prefill, work={"flops": 4 * heads * dim * seen})
+    pair("prefill attention, window", tide_prefill(WINDOW), qwen_prefill, work={"flops": 4 * heads * dim * inside},
+         their_work={"flops": 4 * heads * dim * seen})
+
+    # Projections: bf16 library products against the FP8 kernel (its peak taken as twice the bf16 one).
+    for rows, label in ((batch, "decode"), (tokens, "prefill")):
+        for name, weight, bias, q8, q8s in (("qkv", w.qkv, w.qkv_bias, q.qkv, q.qkv_scale), ("o", w.o, None, q.o, q.o_scale),
+                                            ("gate_up", w.gate_up, None, q.gate_up, q.gate_up_scale),
+                                            ("down", w.down, None, q.down, q.down_scale)):
+            n, k = weight.shape
+            x = bf16(rows, k)
+            x8 = qwen._quantize(x)
+            pair(f"{label} {name} projection", lambda: tide._linear(x, weight, bias),
+                 lambda: qwen._gemm(x8, q8, q8s, rows, k),
+                 work={"bytes_": 2 * (n * k + rows * (n + k)), "flops": 2 * rows * n * k},
+                 their_work={"bytes_": n * k + rows * (2 * n + k), "flops": 2 * rows * n * k, "tensor": 2 * tensor})
+        qkv = bf16(rows, w.qkv.shape[0])
+        pos = (lengths - 1) if label == "decode" else torch.arange(prompt_len, dtype=torch.int32, device=device).repeat(prompts)
+        own = None if label == "decode" else torch.arange(prompts, dtype=torch.int32, device=device).repeat_interleave(prompt_len)
+        tab, q_out = (tables, queries) if label == "decode" else (tables_p, queries_p)
+        pair(f"{label} q/k norm, mix, page write",
+             lambda: qkv_norm_mix_write(qkv, q_out, tide.key_blocks[0], tide.value_blocks[0], pos, own, tab, q_heads=heads,
+                                        kv_heads=kv, dim=dim, value_dim=dim, unit_norm=True, eps=1e-6,
+                                        temperature=layer.temperature, v_first=qkv[:, (heads + kv) * dim:], lam=0.5,
+                                        status=tide.status),
+             lambda: qwen._qkv_post(0, q, qkv, q_out, pos, own, tab, rows, tab.shape[0]),
+             work={"bytes_": 4 * rows * w.qkv.shape[0]})
+        x32, y = torch.randn(rows, width, device=device), bf16(rows, width)
+        xb = x32.to(torch.bfloat16)
+        pair(f"{label} residual sum + norm", lambda: sum_rms_norm(x32, y, w.norm1, eps=1e-6, alpha=2.0, weight_offset=1.0),
+             lambda: qwen._norm(xb, q.input_norm, y, quantize=True), work={"bytes_": rows * width * 12},
+             their_work={"bytes_": rows * width * 7})
+        gate_up = bf16(rows, 2 * ff)
+        pair(f"{label} gate", lambda: clamped_glu(gate_up, limit=7.0, slope=1.702, up_offset=1.0),
+             lambda: qwen._silu_mul_quantized(gate_up, rows), work={"bytes_": rows * ff * 6},
+             their_work={"bytes_": rows * ff * 5})
+        ids = torch.randint(0, vocab, (rows,), device=device)
+        pair(f"{label} embedding",
+             lambda: embed_tokens(ids, tide.weights.embed, pos, own, tab, scale=2.0, page=page, num_pages=tide.total_pages,
+                                  bigram=tide.weights.bigram, mul_prev=31, mul_cur=7, history=tide.history,
+                                  frequencies=tide.weights.frequencies, status=tide.status),
+             lambda: qwen.weights.embedding.index_select(0, ids), work={"bytes_": rows * width * 10},
+             their_work={"bytes_": rows * width * 4})
+        del qkv, x32, y, xb, gate_up
+    final = bf16(batch, width)
+    pair("lm_head + greedy", lambda: tide.lm_head_argmax(final, tide.weights.head), lambda: qwen.greedy_tokens(final),
+         work={"bytes_": 2 * vocab * width})
+    tide.check_status()
+    qwen.check_status()
+    return out
+
+
+def run(device, hbm: float, tensor: float, *, sizes=tuple(SIZES), batch: int = 64, context: int = 2048, prompts: int = 8,
+        prompt_len: int = 2048, steps: int = 50) -> dict:
+    result = {"layers": LAYERS, "window": WINDOW, "decode_batch": batch, "decode_context": context,
+              "prefill": f"{prompts} x {prompt_len}", "hbm_gb_s": hbm, "bf16_tflop_s": tensor, "sizes": {}}
+    for name in sizes:
+        width, heads, kv, dim, ff, vocab = size = SIZES[name]
+        pages = max(batch * (-(-(context + steps + 16) // 16)), prompts * (-(-prompt_len // 16))) + 8
+        options = dict(num_pages=pages, max_batch=batch, max_context=context + steps + 64)
+        shape = TidelornShape.from_config(tidelorn_config(*size))
+        tide = TidelornRunner(TidelornWeights.random(shape, device), kv_init="normal", **options)
+        entry = {"tidelorn": _throughput(tide, vocab, batch, context, prompts, prompt_len, steps, device)}
+        tide.release_graphs()
+        q_shape = Qwen3Shape(layers=LAYERS, hidden=width, q_heads=heads, kv_heads=kv, head_dim=dim, intermediate=ff,
+                             vocab=vocab)
+        qwen = Qwen3DecodeRunner(Qwen3Weights(q_shape, device), kv_init="normal", **options)
+        entry["qwen3_fp8"] = _throughput(qwen, vocab, batch, context, prompts, prompt_len, steps, device)
+        qwen.release_graphs()
+        entry["kernels"] = _kernels(size, tide, qwen, batch, context, prompts, prompt_len, hbm, tensor, device)
+        result["sizes"][name] = entry
+        del tide, qwen
+        gc.collect()
+        torch.cuda.empty_cache()
+    return result

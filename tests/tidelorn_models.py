@@ -91,10 +91,16 @@ def make_tokens(config: dict, count: int, seed: int) -> list[int]:
     return torch.randint(0, config["vocab"], (count,), generator=torch.Generator().manual_seed(seed)).tolist()
 
 
-def logit_error(got: torch.Tensor, want: torch.Tensor) -> float:
-    """Largest row error: root mean square of the centred difference over the vocabulary, in units of the spread
+def logit_errors(got: torch.Tensor, want: torch.Tensor) -> torch.Tensor:
+    """Error of every row: root mean square of the centred difference over the vocabulary, in units of the spread
     of the expected logits."""
 
     difference = got.double().cpu() - want.double()
     difference = difference - difference.mean(dim=-1, keepdim=True)
-    return float(difference.square().mean(dim=-1).sqrt().max() / want.double().std())
+    return difference.square().mean(dim=-1).sqrt() / want.double().std()
+
+
+def logit_error(got: torch.Tensor, want: torch.Tensor) -> float:
+    """Largest row error."""
+
+    return float(logit_errors(got, want).max())
