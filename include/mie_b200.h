@@ -490,12 +490,13 @@ int mie_tp_reduce_rms_norm(const mie_tp_peers_t* peers, int32_t tp, int32_t rank
  *   history [num_blocks, block_size] int32: token ids by page slot, one more
  *     paged cache tensor under the same block tables; every call stores its
  *     own ids there.
- *   frequencies [ceil(width / 2)] float64: entries 2i / 2i + 1 get sin / cos of
- *     positions[t] * frequencies[i].
+ *   turns [ceil(width / 2)][2] fp32: entries 2i / 2i + 1 get sin / cos of
+ *     2 pi * positions[t] * (turns[i][0] + turns[i][1]), a rounded number and
+ *     its remainder (exact for positions below 2^24).
  * token_to_sequence may be NULL (token t is block-table row t).
  */
 int mie_embed_tokens(mie_index_t ids, const void* table, int64_t vocab, float scale, const void* bigram,
-                     int64_t buckets, int64_t mul_prev, int64_t mul_cur, const double* frequencies,
+                     int64_t buckets, int64_t mul_prev, int64_t mul_cur, const float* turns,
                      int32_t* history, mie_index_t positions, mie_index_t token_to_sequence,
                      mie_index_t block_tables, float* out32, void* out, int32_t tokens, int32_t width,
                      int32_t dtype, int32_t block_size, int32_t num_blocks, int32_t table_rows,

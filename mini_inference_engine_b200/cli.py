@@ -81,7 +81,7 @@ def run_trace(args: argparse.Namespace) -> int:
     page = 16
     pages = -(-max(args.max_tokens, 1) // page) + 256  # every live request may leave one page partly filled
     runner = load_runner(args.model, dtype=DTYPES[args.dtype], num_pages=pages, max_batch=8,
-                         max_context=max(args.max_tokens, page))
+                         max_context=args.max_tokens + page)
     session = TraceSession(runner)
     for line in sys.stdin:
         if not line.strip():

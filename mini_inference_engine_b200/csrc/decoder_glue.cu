@@ -114,7 +114,7 @@ struct EmbedParams {
   float scale;
   const void* bigram;         // [buckets + 1][width] or null; the last row is for a sequence's first token
   long long buckets, mul_prev, mul_cur;
-  const double* frequencies;  // [ceil(width / 2)] radians per position, or null
+  const float2* turns;        // [ceil(width / 2)] turns per position as a rounded fp32 part and its remainder, or null
   int* history;               // [num_pages][page] token ids, or null (needed by the bigram part)
   Placement place;
   float* out32;
@@ -122,7 +122,16 @@ struct EmbedParams {
   int tokens, width;
 };
 
-template <typename T>
+// sin and cos of position * turns * 2 pi: the whole turns of the product are taken off with its rounding error kept,
+// so that a far position has a full fp32 angle.
+__device__ __forceinline__ void turn_sincos(float position, float2 turns, float* sine, float* cosine) {
+  const float product = position * turns.x;
+  const float error = fmaf(position, turns.x, -product);
+  const float rest = (product - rintf(product)) + fmaf(position, turns.y, error);
+  sincospif(2.f * rest, sine, cosine);
+}
+
+template <typename T, int VEC>
 __global__ void embed_kernel(EmbedParams p) {
   chain_wait();
   chain_release();
@@ -164,25 +173,35 @@ __global__ void embed_kernel(EmbedParams p) {
   const T* row = reinterpret_cast<const T*>(p.table) + id * p.width;
   float* out32 = p.out32 + (long long)t * p.width;
   T* out = p.out == nullptr ? nullptr : reinterpret_cast<T*>(p.out) + (long long)t * p.width;
-  for (int pair = threadIdx.x; 2 * pair < p.width; pair += blockDim.x) {
-    float add[2] = {0.f, 0.f};
-    if (p.frequencies != nullptr) {
-      // The angle is reduced to one turn in double precision, so a far position keeps a full fp32 angle.
-      constexpr double kTurn = 6.283185307179586476925;
-      double angle = (double)pos * p.frequencies[pair];
-      angle -= kTurn * rint(angle / kTurn);
-      sincosf((float)angle, &add[0], &add[1]);
-    }
+  const float position = (float)pos;
+  for (int c = threadIdx.x * VEC; c < p.width; c += blockDim.x * VEC) {
+    float v[VEC];
+    Vec<T, VEC>::load(row + c, v);
 #pragma unroll
-    for (int i = 0; i < 2; ++i) {
-      const int c = 2 * pair + i;
-      if (c >= p.width) break;
-      float v = to_float<T>(row[c]) * p.scale;
-      if (bigram_row != nullptr) v += to_float<T>(bigram_row[c]);
-      v += add[i];
-      out32[c] = v;
-      if (out != nullptr) out[c] = from_float<T>(v);
+    for (int j = 0; j < VEC; ++j) v[j] *= p.scale;
+    if (bigram_row != nullptr) {
+      float b[VEC];
+      Vec<T, VEC>::load(bigram_row + c, b);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) v[j] += b[j];
     }
+    if (p.turns != nullptr) {
+      if (VEC == 1) {
+        float sine, cosine;
+        turn_sincos(position, p.turns[c / 2], &sine, &cosine);
+        v[0] += c % 2 == 0 ? sine : cosine;
+      } else {
+#pragma unroll
+        for (int j = 0; j + 1 < VEC; j += 2) {
+          float sine, cosine;
+          turn_sincos(position, p.turns[(c + j) / 2], &sine, &cosine);
+          v[j] += sine;
+          v[j + 1] += cosine;
+        }
+      }
+    }
+    Vec<float, VEC>::store(out32 + c, v);
+    if (out != nullptr) Vec<T, VEC>::store(out + c, v);
   }
 }
 
@@ -259,7 +278,7 @@ __global__ void __launch_bounds__(1024) sum_norm_kernel(SumNormParams p) {
 }
 
 // ---------------------------------------------------------------------------
-// Between the merged projection and attention: one warp per (token, head slot).
+// Between the merged projection and attention: LANES lanes per (token, head slot).
 //   q: optional unit-RMS norm, optional position-dependent temperature, to q_out
 //   k: optional unit-RMS norm, to its page
 //   v: optional blend with another layer's values of the same token, to its page
@@ -282,16 +301,16 @@ struct QkvMixParams {
   Placement place;
 };
 
-template <typename T, int VEC>
+template <typename T, int VEC, int LANES>
 __global__ void qkv_mix_kernel(QkvMixParams p) {
   chain_wait();
   chain_release();
-  const long long warp = ((long long)blockIdx.x * blockDim.x + threadIdx.x) >> 5;
-  const int lane = threadIdx.x & 31;
+  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / LANES;
+  const int lane = threadIdx.x % LANES;
   const int slots = p.q_heads + 2 * p.kv_heads;
-  if (warp >= (long long)p.tokens * slots) return;
-  const long long t = warp / slots;
-  const int h = (int)(warp % slots);
+  const bool live = item < (long long)p.tokens * slots;  // idle lanes stay for the shuffles of their warp
+  const long long t = live ? item / slots : 0;
+  const int h = live ? (int)(item % slots) : 0;
   const bool is_q = h < p.q_heads, is_v = h >= p.q_heads + p.kv_heads;
   const int kvh = is_v ? h - p.q_heads - p.kv_heads : h - p.q_heads;
   const int n = is_v ? p.vdim : p.dim;
@@ -300,16 +319,21 @@ __global__ void qkv_mix_kernel(QkvMixParams p) {
   const T* src = reinterpret_cast<const T*>(p.qkv) + t * p.ld + offset;
   const long long pos = p.place.positions.at(t);
   float factor = 1.f;
-  if (!is_v && p.unit_norm) {
+  if (p.unit_norm) {
     float ss = 0.f;
-    for (int c = lane * VEC; c < n; c += 32 * VEC) {
-      float v[VEC];
-      Vec<T, VEC>::load(src + c, v);
+    if (!is_v) {
+      for (int c = lane * VEC; c < n; c += LANES * VEC) {
+        float v[VEC];
+        Vec<T, VEC>::load(src + c, v);
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) ss += v[j] * v[j];
+        for (int j = 0; j < VEC; ++j) ss += v[j] * v[j];
+      }
     }
-    factor = 1.f / sqrtf(warp_sum(ss) / (float)n + p.eps);
+#pragma unroll
+    for (int o = LANES / 2; o > 0; o >>= 1) ss += __shfl_xor_sync(0xffffffffu, ss, o);
+    if (!is_v) factor = 1.f / sqrtf(ss / (float)n + p.eps);
   }
+  if (!live) return;
   if (is_q && p.temp_every > 0) {
     const long long block = (pos + 1) / p.temp_every;
     factor *= 1.f + p.temp_coef * logf((float)(block + 1));
@@ -327,7 +351,7 @@ __global__ void qkv_mix_kernel(QkvMixParams p) {
   const T* first = is_v && p.v_first != nullptr
                        ? reinterpret_cast<const T*>(p.v_first) + t * p.ld_first + (long long)kvh * p.vdim
                        : nullptr;
-  for (int c = lane * VEC; c < n; c += 32 * VEC) {
+  for (int c = lane * VEC; c < n; c += LANES * VEC) {
     float v[VEC];
     Vec<T, VEC>::load(src + c, v);
     if (first != nullptr) {
@@ -398,14 +422,13 @@ int launch_sum_norm(const SumNormParams& p, bool vec, cudaStream_t stream) {
 }
 
 template <typename T>
-int launch_qkv_mix(const QkvMixParams& p, bool vec, cudaStream_t stream) {
-  const long long warps = (long long)p.tokens * (p.q_heads + 2 * p.kv_heads);
-  const int threads = 256;
-  const dim3 grid((unsigned)((warps * 32 + threads - 1) / threads));
-  if (vec)
-    MIE_CUDA(launch_chained(qkv_mix_kernel<T, 4>, grid, dim3(threads), 0, stream, p));
-  else
-    MIE_CUDA(launch_chained(qkv_mix_kernel<T, 1>, grid, dim3(threads), 0, stream, p));
+int launch_qkv_mix(const QkvMixParams& p, int vec, cudaStream_t stream) {
+  const long long slots = (long long)p.tokens * (p.q_heads + 2 * p.kv_heads);
+  const int threads = 256, lanes = vec == 8 ? 16 : 32;
+  const dim3 grid((unsigned)((slots * lanes + threads - 1) / threads)), block(threads);
+  MIE_CUDA(vec == 8   ? launch_chained(qkv_mix_kernel<T, 8, 16>, grid, block, 0, stream, p)
+           : vec == 4 ? launch_chained(qkv_mix_kernel<T, 4, 32>, grid, block, 0, stream, p)
+                      : launch_chained(qkv_mix_kernel<T, 1, 32>, grid, block, 0, stream, p));
   MIE_LAUNCH_CHECK("qkv_mix_kernel");
   return MIE_OK;
 }
@@ -435,7 +458,7 @@ using namespace mie;
   MIE_CHECK_ARG((dtype) == MIE_DTYPE_BF16 || (dtype) == MIE_DTYPE_F32, "activations are bf16 or fp32")
 
 extern "C" int mie_embed_tokens(mie_index_t ids, const void* table, int64_t vocab, float scale, const void* bigram,
-                                int64_t buckets, int64_t mul_prev, int64_t mul_cur, const double* frequencies,
+                                int64_t buckets, int64_t mul_prev, int64_t mul_cur, const float* turns,
                                 int32_t* history, mie_index_t positions, mie_index_t token_to_sequence,
                                 mie_index_t block_tables, float* out32, void* out, int32_t tokens, int32_t width,
                                 int32_t dtype, int32_t block_size, int32_t num_blocks, int32_t table_rows,
@@ -457,7 +480,7 @@ extern "C" int mie_embed_tokens(mie_index_t ids, const void* table, int64_t voca
   p.buckets = buckets;
   p.mul_prev = mul_prev;
   p.mul_cur = mul_cur;
-  p.frequencies = frequencies;
+  p.turns = reinterpret_cast<const float2*>(turns);
   p.history = history;
   p.place = placement(positions, token_to_sequence, block_tables, block_size, num_blocks, table_rows, table_width,
                       status);
@@ -465,12 +488,17 @@ extern "C" int mie_embed_tokens(mie_index_t ids, const void* table, int64_t voca
   p.out = out;
   p.tokens = tokens;
   p.width = width;
-  int threads = ((width + 1) / 2 + 31) / 32 * 32;
+  MIE_CHECK_ARG(aligned(turns, 8), "the turns must be 8-byte aligned pairs");
+  const bool vec = width % 8 == 0 && aligned(table, 16) && aligned(bigram, 16) && aligned(out32, 16) && aligned(out, 16);
+  int threads = ((vec ? width / 8 : width) + 31) / 32 * 32;
   if (threads > 256) threads = 256;
+  const dim3 grid(tokens), block(threads);
   if (dtype == MIE_DTYPE_BF16)
-    MIE_CUDA(launch_chained(embed_kernel<__nv_bfloat16>, dim3(tokens), dim3(threads), 0, (cudaStream_t)stream, p));
+    MIE_CUDA(vec ? launch_chained(embed_kernel<__nv_bfloat16, 8>, grid, block, 0, (cudaStream_t)stream, p)
+                 : launch_chained(embed_kernel<__nv_bfloat16, 1>, grid, block, 0, (cudaStream_t)stream, p));
   else
-    MIE_CUDA(launch_chained(embed_kernel<float>, dim3(tokens), dim3(threads), 0, (cudaStream_t)stream, p));
+    MIE_CUDA(vec ? launch_chained(embed_kernel<float, 8>, grid, block, 0, (cudaStream_t)stream, p)
+                 : launch_chained(embed_kernel<float, 1>, grid, block, 0, (cudaStream_t)stream, p));
   MIE_LAUNCH_CHECK("embed_kernel");
   return MIE_OK;
 }
@@ -517,14 +545,20 @@ extern "C" int mie_qkv_norm_mix_write(const void* qkv, int64_t ld, const void* v
   p.q_out = q_out;
   p.key_blocks = (char*)key_blocks.ptr;
   p.value_blocks = (char*)value_blocks.ptr;
-  bool vec = dim % 4 == 0 && value_dim % 4 == 0 && ld % 4 == 0 && ld_first % 4 == 0;
+  // Widest vector that every row, stride and address allows.
+  auto fits = [&](int v) {
+    const int bytes = v * (dtype == MIE_DTYPE_BF16 ? 2 : 4) < 16 ? 8 : 16;
+    bool ok = dim % v == 0 && value_dim % v == 0 && ld % v == 0 && ld_first % v == 0 && aligned(qkv, bytes) &&
+              aligned(v_first, bytes) && aligned(q_out, bytes) && aligned(key_blocks.ptr, bytes) &&
+              aligned(value_blocks.ptr, bytes);
+    for (int i = 0; i < 3; ++i) ok = ok && key_blocks.stride[i] % v == 0 && value_blocks.stride[i] % v == 0;
+    return ok;
+  };
   for (int i = 0; i < 3; ++i) {
     p.kb_s[i] = key_blocks.stride[i];
     p.vb_s[i] = value_blocks.stride[i];
-    vec = vec && p.kb_s[i] % 4 == 0 && p.vb_s[i] % 4 == 0;
   }
-  vec = vec && aligned(qkv, 16) && aligned(v_first, 8) && aligned(q_out, 16) && aligned(key_blocks.ptr, 16) &&
-        aligned(value_blocks.ptr, 16) && (dtype == MIE_DTYPE_BF16 || aligned(v_first, 16));
+  const int vec = fits(8) ? 8 : fits(4) ? 4 : 1;
   p.tokens = tokens;
   p.q_heads = q_heads;
   p.kv_heads = kv_heads;

@@ -7,13 +7,25 @@ key heads are normalised, a query temperature, value mixing, the limits of a gat
 
 from __future__ import annotations
 
+import math
+
 import torch
 
 from ... import _lib
 
 
+def sinusoid_turns(width: int, base: float, device: torch.device) -> torch.Tensor:
+    """``[ceil(width / 2), 2]`` fp32: base^(-2i / width) / 2 pi, the turns of entry pair i per position, as a
+    rounded number and its remainder."""
+
+    turns = torch.tensor([base ** (-2.0 * i / width) / (2.0 * math.pi) for i in range((width + 1) // 2)],
+                         dtype=torch.float64)
+    high = turns.float()
+    return torch.stack((high, (turns - high.double()).float()), dim=1).contiguous().to(device)
+
+
 def embed_tokens(ids, table, positions, token_to_sequence, block_tables, *, scale: float, page: int, num_pages: int,
-                 bigram=None, mul_prev: int = 0, mul_cur: int = 0, history=None, frequencies=None,
+                 bigram=None, mul_prev: int = 0, mul_cur: int = 0, history=None, turns=None,
                  status: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
     """``(fp32 rows, activation rows)`` of table[id] * scale (+ bigram row) (+ sinusoid).  ``history``
     (``[pages, page]`` int32) is the paged record of token ids the bigram part reads a predecessor from."""
@@ -23,7 +35,7 @@ def embed_tokens(ids, table, positions, token_to_sequence, block_tables, *, scal
     out = out32 if table.dtype == torch.float32 else torch.empty(tokens, width, dtype=table.dtype, device=table.device)
     _lib.check(_lib.load().mie_embed_tokens(
         _lib.index_arg(ids), _lib.ptr(table), int(table.shape[0]), float(scale), _lib.ptr(bigram),
-        0 if bigram is None else int(bigram.shape[0]) - 1, int(mul_prev), int(mul_cur), _lib.ptr(frequencies),
+        0 if bigram is None else int(bigram.shape[0]) - 1, int(mul_prev), int(mul_cur), _lib.ptr(turns),
         _lib.ptr(history), _lib.index_arg(positions), _lib.index_arg(token_to_sequence), _lib.index_arg(block_tables),
         _lib.ptr(out32), None if out is out32 else _lib.ptr(out), tokens, width, _lib.DTYPE_CODES[table.dtype], page,
         num_pages, int(block_tables.shape[0]), int(block_tables.shape[1]), _lib.ptr(status),
@@ -81,4 +93,4 @@ def clamped_glu(gate_up, *, limit: float, slope: float, up_offset: float) -> tor
     return out
 
 
-__all__ = ["clamped_glu", "embed_tokens", "qkv_norm_mix_write", "sum_rms_norm"]
+__all__ = ["clamped_glu", "embed_tokens", "qkv_norm_mix_write", "sinusoid_turns", "sum_rms_norm"]

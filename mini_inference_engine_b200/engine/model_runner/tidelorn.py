@@ -24,7 +24,7 @@ from dataclasses import dataclass
 
 import torch
 
-from ..kernels.decoder_glue import clamped_glu, embed_tokens, qkv_norm_mix_write, sum_rms_norm
+from ..kernels.decoder_glue import clamped_glu, embed_tokens, qkv_norm_mix_write, sinusoid_turns, sum_rms_norm
 from ..kv_cache.sink_attention import (
     attention_rows,
     sink_decode_attention,
@@ -191,8 +191,7 @@ class TidelornWeights:
                 torch.cat([fetch(f"l{i}.mlp.gate"), fetch(f"l{i}.mlp.up")]) if dense else None,
                 fetch(f"l{i}.mlp.down") if dense else None, fetch(f"l{i}.norm2") if dense else None))
         self.final_norm, self.head = fetch("final.norm"), fetch("head")
-        frequencies = [SINUSOID_BASE ** (-2.0 * i / shape.width) for i in range((shape.width + 1) // 2)]
-        self.frequencies = torch.tensor(frequencies, dtype=torch.float64, device=device)
+        self.turns = sinusoid_turns(shape.width, SINUSOID_BASE, device)
 
     @classmethod
     def random(cls, shape: TidelornShape, device: torch.device, *, seed: int = 0,
@@ -330,7 +329,7 @@ class TidelornRunner(PagedStepRunner):
         x32, x = embed_tokens(input_ids, weights.embed, positions, token_to_sequence, block_tables,
                               scale=shape.embed_scale, page=shape.page, num_pages=self.total_pages,
                               bigram=weights.bigram, mul_prev=shape.mul_prev, mul_cur=shape.mul_cur,
-                              history=self.history, frequencies=weights.frequencies, status=self.status)
+                              history=self.history, turns=weights.turns, status=self.status)
         v_first, plans = None, {}
         norm = dict(eps=shape.eps, alpha=shape.alpha, weight_offset=NORM_WEIGHT_OFFSET)
         for index, (layer, w) in enumerate(zip(shape.layers, weights.layers)):

@@ -216,7 +216,7 @@ def _kernels(size, tide: TidelornRunner, qwen: Qwen3DecodeRunner, batch, context
         pair(f"{label} embedding",
              lambda: embed_tokens(ids, tide.weights.embed, pos, own, tab, scale=2.0, page=page, num_pages=tide.total_pages,
                                   bigram=tide.weights.bigram, mul_prev=31, mul_cur=7, history=tide.history,
-                                  frequencies=tide.weights.frequencies, status=tide.status),
+                                  turns=tide.weights.turns, status=tide.status),
              lambda: qwen.weights.embedding.index_select(0, ids), work={"bytes_": rows * width * 10},
              their_work={"bytes_": rows * width * 4})
         del qkv, x32, y, xb, gate_up

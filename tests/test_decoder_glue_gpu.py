@@ -9,6 +9,7 @@ from mini_inference_engine_b200.engine.kernels.decoder_glue import (
     clamped_glu,
     embed_tokens,
     qkv_norm_mix_write,
+    sinusoid_turns,
     sum_rms_norm,
 )
 from oracle import tidelorn_model as plain
@@ -44,7 +45,7 @@ def test_embedding_parts_and_previous_token(dtype, width, device):
               1: torch.randint(0, vocab, (9,), generator=generator).tolist()}
     tables = torch.tensor([[3, 7, 1, 9, 5], [2, 8, 0, -1, -1]], dtype=torch.int32)
     history = torch.full((10, page), -1, dtype=torch.int32, device=device)
-    frequencies = torch.tensor([10000.0 ** (-2.0 * i / width) for i in range((width + 1) // 2)], dtype=torch.float64)
+    turns = sinusoid_turns(width, 10000.0, device)
     want = {}
     for row, ids in tokens.items():
         rows = plain.bigram_rows(ids, buckets, 31, 7)
@@ -65,7 +66,7 @@ def test_embedding_parts_and_previous_token(dtype, width, device):
                               torch.tensor(positions, dtype=torch.int32, device=device),
                               torch.tensor(owners, dtype=torch.int32, device=device), tables.to(device), scale=1.75,
                               page=page, num_pages=10, bigram=bigram.to(device), mul_prev=31, mul_cur=7,
-                              history=history, frequencies=frequencies.to(device), status=word)
+                              history=history, turns=turns, status=word)
         close(x32, torch.cat(expected))
         close(x, torch.cat(expected))
     assert int(word.item()) == 0 and at == {0: 19, 1: 9}
@@ -75,7 +76,7 @@ def test_embedding_far_positions_large_ids_and_bare_table(device):
     vocab, width = 140_000, 48
     table = torch.randn(vocab, width, generator=torch.Generator().manual_seed(1))
     bigram = torch.randn(1_000_004, width, generator=torch.Generator().manual_seed(2))
-    frequencies = torch.tensor([10000.0 ** (-2.0 * i / width) for i in range(width // 2)], dtype=torch.float64)
+    turns = sinusoid_turns(width, 10000.0, device)
     word, position = status(device), 131_071
     tables = torch.arange(8192, dtype=torch.int32, device=device).unsqueeze(0)
     history = torch.zeros(8192, 16, dtype=torch.int32, device=device)
@@ -85,7 +86,7 @@ def test_embedding_far_positions_large_ids_and_bare_table(device):
     multipliers = (2_000_003, 1_999_993)  # products beyond 32 bits
     x32, _ = embed_tokens(ids, table.to(device), place, None, tables, scale=0.5, page=16, num_pages=8192,
                           bigram=bigram.to(device), mul_prev=multipliers[0], mul_cur=multipliers[1], history=history,
-                          frequencies=frequencies.to(device), status=word)
+                          turns=turns, status=word)
     row = (139_998 * multipliers[0] + 139_999 * multipliers[1]) % 1_000_003
     want = table[139_999].double() * 0.5 + bigram[row].double() + plain.sinusoid(torch.tensor([position]), width)[0]
     close(x32[0], want)

@@ -312,3 +312,19 @@ def test_command_line_replays_and_generates(model_folder, device):
     assert done.returncode == 0, done.stderr[-2000:]
     lines = [json.loads(line) for line in done.stdout.splitlines() if line.startswith("{")]
     assert [line["tokens"] for line in lines] == [tokens[:4] for *_, tokens in requests]
+
+
+def test_the_registry_serves_the_other_design_too(tmp_path, device):
+    """A Qwen3 configuration through the same registry, batcher and runner interface (seeded weights): scheduled
+    generation gives the tokens of its own ``generate``."""
+
+    (tmp_path / "config.json").write_text(json.dumps({
+        "architectures": ["Qwen3ForCausalLM"], "num_hidden_layers": 2, "hidden_size": 512, "num_attention_heads": 4,
+        "num_key_value_heads": 2, "head_dim": 128, "intermediate_size": 1024, "vocab_size": 2048,
+        "rms_norm_eps": 1e-6, "rope_theta": 5e6}))
+    runner = load_runner(tmp_path, random_seed=36, num_pages=32, max_batch=2, max_context=128)
+    prompt = torch.randint(0, 2048, (37,), generator=torch.Generator().manual_seed(1)).tolist()
+    batcher = ContinuousBatcher(runner)
+    batcher.submit("a", prompt, 3)
+    assert batcher.run()["a"] == runner.generate([prompt], 3)[0]
+    runner.release_graphs()
