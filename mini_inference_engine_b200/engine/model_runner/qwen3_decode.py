@@ -39,6 +39,7 @@ from .peer_exchange import PeerExchange
 from .step_runner import (
     DEFAULT_DECODE_BUCKETS,
     PADDING,
+    PLAN_SLOTS,
     DecodeBuffers,
     MixedBuffers,
     PagedStepRunner,
@@ -47,11 +48,6 @@ from .step_runner import (
 from ..kv_cache.fp8_kv import Fp8KvPool, launch_decode_attention_kv8
 from ..kv_cache.triton_flash_prefill import launch_flash_prefill
 from ..kv_cache.triton_paged_attention import decode_scratch, launch_decode_attention
-
-
-# A decode work plan carries 64 work counters, one per attention launch that reuses it; deeper models
-# rebuild the plan every 64 layers.
-PLAN_SLOTS = 64
 
 
 @dataclass(frozen=True)

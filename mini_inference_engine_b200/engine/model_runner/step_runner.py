@@ -14,6 +14,9 @@ import torch
 from ... import _lib
 
 
+# A decode work plan carries 64 work counters, one per attention launch that reuses it; deeper models
+# rebuild the plan every 64 layers.
+PLAN_SLOTS = 64
 LM_HEAD_MAX_ROWS = 256  # rows one mie_lm_head_argmax call takes
 DEFAULT_DECODE_BUCKETS = (1, 2, 4, 8, 16, 32, 64, 128, 256)
 
@@ -557,5 +560,5 @@ class PagedStepRunner:
         _lib.raise_for_status(self.status)
 
 
-__all__ = ["DEFAULT_DECODE_BUCKETS", "DecodeBuffers", "MixedBuffers", "PADDING", "PagedStepRunner", "eager_step",
-           "select_bucket"]
+__all__ = ["DEFAULT_DECODE_BUCKETS", "DecodeBuffers", "LM_HEAD_MAX_ROWS", "MixedBuffers", "PADDING", "PLAN_SLOTS",
+           "PagedStepRunner", "eager_step", "select_bucket"]

@@ -34,12 +34,11 @@ from ..kv_cache.sink_attention import (
 )
 from ..kv_cache.triton_paged_attention import decode_scratch
 from ... import _lib
-from .step_runner import PagedStepRunner
+from .step_runner import PLAN_SLOTS, PagedStepRunner
 
 SINUSOID_BASE = 10000.0
 GATE_SLOPE = 1.702
 UP_OFFSET = 1.0
-PLAN_SLOTS = 64  # work counters of one decode work plan
 NORM_WEIGHT_OFFSET = 1.0  # norm weights are stored as their deviation from one
 
 

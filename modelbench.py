@@ -22,7 +22,7 @@ from mini_inference_engine_b200.engine.kernels.decoder_glue import (
 )
 from mini_inference_engine_b200.engine.kv_cache.sink_attention import sink_decode_attention, sink_prefill_attention
 from mini_inference_engine_b200.engine.kv_cache.triton_flash_prefill import launch_flash_prefill
-from mini_inference_engine_b200.engine.kv_cache.triton_paged_attention import launch_decode_attention
+from mini_inference_engine_b200.engine.kv_cache.triton_paged_attention import decode_scratch, launch_decode_attention
 from mini_inference_engine_b200.engine.model_runner.qwen3_decode import Qwen3DecodeRunner, Qwen3Shape, Qwen3Weights
 from mini_inference_engine_b200.engine.model_runner.tidelorn import TidelornRunner, TidelornShape, TidelornWeights
 
@@ -228,10 +228,43 @@ def _kernels(size, tide: TidelornRunner, qwen: Qwen3DecodeRunner, batch, context
     return out
 
 
+# Head sizes that are not two 64-dim boxes: key size, value size.
+HEAD_SIZES = ((64, 64), (96, 96), (192, 128), (256, 256))
+
+
+def head_sizes(device, hbm: float, tensor: float, *, heads: int = 32, kv: int = 8, batch: int = 64, context: int = 2048,
+               prompts: int = 4, prompt_len: int = 2048) -> dict:
+    """The two streaming attention kernels at other head sizes (whole prefix)."""
+
+    flush, out = Flusher(device), {}
+    pages = batch * (context // 16) + 8
+    tables = _tables(batch, context // 16, pages, device)
+    lengths = torch.full((batch,), context, dtype=torch.int32, device=device)
+    cu = torch.arange(prompts + 1, dtype=torch.int32, device=device) * prompt_len
+    status = torch.zeros(1, dtype=torch.int32, device=device)
+    sinks = torch.zeros(heads, device=device)
+    for dim, vdim in HEAD_SIZES:
+        keys, values = (torch.randn(pages, kv, 16, n, device=device).to(torch.bfloat16) for n in (dim, vdim))
+        scratch = decode_scratch(batch, heads, kv, vdim, batch * context, device)
+        common = dict(scale=dim ** -0.5, sinks=sinks, status=status)
+        rows = prompts * prompt_len
+        query, result = (torch.randn(rows, heads, n, device=device).to(torch.bfloat16) for n in (dim, vdim))
+        decode = flush.median_us(lambda: sink_decode_attention(query[:batch], result[:batch], keys, values, tables,
+                                                               lengths, scratch=scratch, **common))
+        prefill = flush.median_us(lambda: sink_prefill_attention(query, result, keys, values, tables[:prompts], cu,
+                                                                 lengths[:prompts], max_query_len=prompt_len, **common))
+        flops = 2 * heads * (dim + vdim) * prompts * prompt_len * (prompt_len + 1) / 2
+        out[f"{dim}/{vdim}"] = {
+            "decode": _row(decode, bytes_=batch * context * kv * (dim + vdim) * 2, hbm=hbm, tensor=tensor),
+            "prefill": _row(prefill, flops=flops, hbm=hbm, tensor=tensor)}
+    return out
+
+
 def run(device, hbm: float, tensor: float, *, sizes=tuple(SIZES), batch: int = 64, context: int = 2048, prompts: int = 8,
         prompt_len: int = 2048, steps: int = 50) -> dict:
     result = {"layers": LAYERS, "window": WINDOW, "decode_batch": batch, "decode_context": context,
-              "prefill": f"{prompts} x {prompt_len}", "hbm_gb_s": hbm, "bf16_tflop_s": tensor, "sizes": {}}
+              "prefill": f"{prompts} x {prompt_len}", "hbm_gb_s": hbm, "bf16_tflop_s": tensor, "sizes": {},
+              "head_sizes": head_sizes(device, hbm, tensor)}
     for name in sizes:
         width, heads, kv, dim, ff, vocab = size = SIZES[name]
         pages = max(batch * (-(-(context + steps + 16) // 16)), prompts * (-(-prompt_len // 16))) + 8
