@@ -47,7 +47,7 @@ def tidelorn_config(width, heads, kv_heads, dim, ff, vocab, layers=LAYERS, windo
         entries.append({"type": "attention" if index % 2 == 0 else "attention_2", "mixer": mixer,
                         "mlp": {"kind": "dense", "ff": ff, "limit": 7.0}})
     return {"vocab": vocab, "width": width, "norm": {"eps": 1e-6}, "postln_alpha": 2.0, "layers": entries,
-            "embedding": {"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 31, "mul_cur": 7}}}
+            "embedding": {"scale": width ** 0.5, "bigram": {"buckets": 65521, "mul_prev": 8191, "mul_cur": 127}}}
 
 
 def _tables(batch: int, pages_each: int, total: int, device) -> torch.Tensor:
@@ -215,7 +215,7 @@ def _kernels(size, tide: TidelornRunner, qwen: Qwen3DecodeRunner, batch, context
         ids = torch.randint(0, vocab, (rows,), device=device)
         pair(f"{label} embedding",
              lambda: embed_tokens(ids, tide.weights.embed, pos, own, tab, scale=2.0, page=page, num_pages=tide.total_pages,
-                                  bigram=tide.weights.bigram, mul_prev=31, mul_cur=7, history=tide.history,
+                                  bigram=tide.weights.bigram, mul_prev=8191, mul_cur=127, history=tide.history,
                                   turns=tide.weights.turns, status=tide.status),
              lambda: qwen.weights.embedding.index_select(0, ids), work={"bytes_": rows * width * 10},
              their_work={"bytes_": rows * width * 4})

@@ -48,7 +48,7 @@ def test_embedding_parts_and_previous_token(dtype, width, device):
     turns = sinusoid_turns(width, 10000.0, device)
     want = {}
     for row, ids in tokens.items():
-        rows = plain.bigram_rows(ids, buckets, 31, 7)
+        rows = plain.bigram_rows(ids, buckets, 29, 11)
         want[row] = (table[ids].double() * 1.75 + bigram[rows].double()
                      + plain.sinusoid(torch.arange(len(ids)), width))
     word = status(device)
@@ -65,7 +65,7 @@ def test_embedding_parts_and_previous_token(dtype, width, device):
         x32, x = embed_tokens(torch.tensor(ids, device=device), table.to(device),
                               torch.tensor(positions, dtype=torch.int32, device=device),
                               torch.tensor(owners, dtype=torch.int32, device=device), tables.to(device), scale=1.75,
-                              page=page, num_pages=10, bigram=bigram.to(device), mul_prev=31, mul_cur=7,
+                              page=page, num_pages=10, bigram=bigram.to(device), mul_prev=29, mul_cur=11,
                               history=history, turns=turns, status=word)
         close(x32, torch.cat(expected))
         close(x, torch.cat(expected))
