@@ -83,6 +83,7 @@ def _throughput(runner, vocab: int, batch: int, context: int, prompts: int, prom
     page = runner.shape.page
     pages_each = -(-(context + steps + 16) // page)
     buffers = runner.capture(batch, pages_each, advance=True)
+    launches = runner.launches_per_step
     buffers.block_tables.copy_(_tables(batch, pages_each, runner.num_pages, device))
     buffers.input_ids.copy_(torch.randint(0, vocab, (batch,), device=device))
     buffers.sequence_lengths.fill_(context + 1)
@@ -107,7 +108,7 @@ def _throughput(runner, vocab: int, batch: int, context: int, prompts: int, prom
     prefill_ms = _event_ms(prefill, 5, device)
     runner.check_status()
     return {"decode": {"ms_per_step": decode_ms, "tok_per_s": batch / decode_ms * 1e3,
-                       "launches_of_this_library": runner.launches_per_step},
+                       "launches_of_this_library": launches},
             "prefill": {"ms": prefill_ms, "tok_per_s": tokens / prefill_ms * 1e3}}
 
 
