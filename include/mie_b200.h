@@ -45,6 +45,7 @@ extern "C" {
 #define MIE_STATUS_CAPACITY 64       /* work plan did not fit the scratch the caller sized */
 #define MIE_STATUS_NO_TOKEN 128      /* greedy sampling saw no candidate for a row; token 0 was written */
 #define MIE_STATUS_BAD_TOKEN 256     /* token id outside the vocabulary (row 0 was used) */
+#define MIE_STATUS_BAD_SLOT 512      /* state slot outside the state buffer (the row was skipped) */
 
 /* Element types of K/V pages, queries and activations. */
 #define MIE_DTYPE_BF16 0
@@ -581,6 +582,119 @@ int mie_sink_prefill_attention(const void* query, int64_t q_token_stride, int64_
                                int32_t kv_heads, int32_t dim, int32_t value_dim, int32_t block_size,
                                int32_t num_blocks, int32_t table_width, int32_t dtype, float scale, int64_t window,
                                const float* sinks, int32_t* status, void* stream);
+
+/* ------------------------------------------------------------------------
+ * Sublayers with a norm before and after, latent attention, recurrent mixers
+ * (activations "T" bf16 or fp32 by `dtype`, as above)
+ * ---------------------------------------------------------------------- */
+
+/*
+ * x += alpha * rms_norm(y) * y_weight (x fp32 in place, y and weights T), then
+ * out = rms_norm(x) * next_weight as T, or x itself as T when next_weight is
+ * NULL; out NULL: only x.  rms_norm(v) = v / sqrt(mean(v^2) + eps).
+ */
+int mie_residual_norm(float* x, int64_t ldx, const void* y, int64_t ldy, const void* y_weight, float alpha,
+                      const void* next_weight, void* out, int64_t ldo, int32_t rows, int32_t cols, int32_t dtype,
+                      float eps, void* stream);
+
+/* out = gelu(in), tanh form, times table[ids[row]][col] when a table is given (row stride ld_table). */
+int mie_gelu(const void* in, int64_t ld_in, mie_index_t ids, const void* table, int64_t ld_table, int64_t vocab,
+             void* out, int64_t ldo, int32_t rows, int32_t cols, int32_t dtype, int32_t* status, void* stream);
+
+/* out = rms_norm(x) * weight * sigmoid(gate). */
+int mie_gated_norm(const void* x, int64_t ldx, const void* gate, int64_t ldg, const void* weight, void* out,
+                   int64_t ldo, int32_t rows, int32_t cols, int32_t dtype, float eps, void* stream);
+
+/* logits <- cap * tanh(logits / cap), in place. */
+int mie_softcap(float* logits, int64_t count, float cap, void* stream);
+
+/*
+ * One merged projection row [q_rank | rank | rot_dim] (row stride ld) ->
+ * rms_norm(first part) * q_weight to q_out, and, with pages, the cached row
+ * [rms_norm(second part) * weight | third part rotated] to the token's slot of
+ * pages [num_blocks][block_size][rank + rot_dim] (strides in elements).
+ * Rotation: entries 2i / 2i + 1 of the first `rotated` ones by the angle
+ * 2 pi * position * (turns[i][0] + turns[i][1]); the rest pass.
+ */
+int mie_latent_norm_write(const void* rows, int64_t ld, int32_t q_rank, int32_t rank, int32_t rot_dim,
+                          int32_t rotated, const void* q_weight, const void* weight, const float* turns,
+                          void* q_out, int64_t ldq, void* pages, int64_t page_stride, int64_t slot_stride,
+                          mie_index_t positions, mie_index_t token_to_sequence, mie_index_t block_tables,
+                          int32_t tokens, int32_t dtype, int32_t block_size, int32_t num_blocks, int32_t table_rows,
+                          int32_t table_width, float eps, int32_t* status, void* stream);
+
+/* The same rotation of [tokens, heads, rot_dim] rows (strided), in place (dst == src) or into dst. */
+int mie_rotate_heads(const void* src, int64_t src_token_stride, int64_t src_head_stride, void* dst,
+                     int64_t dst_token_stride, int64_t dst_head_stride, mie_index_t positions, const float* turns,
+                     int32_t tokens, int32_t heads, int32_t rot_dim, int32_t rotated, int32_t dtype, void* stream);
+
+/*
+ * Spans of cached tokens that packed chunks see through a window, laid end to
+ * end in a buffer of row_capacity rows: request r's tokens from its first
+ * visible one (rounded down to 16) to kv_lens[r], padded to 16 rows.
+ *   spans [2 * requests + 1]: first row per request, first token per request,
+ *     rows in total;  span_lens [requests]: kv_lens counted from the first
+ *     token;  span_table [requests, span_table_width]: the span as 16-token
+ *     pages of the buffer.
+ * mie_latent_gather copies those rows of one cache ([pages][slot][cols]) into
+ * out [rows, cols]; rows past a request's end are zero, rows past the total
+ * are left alone.
+ */
+int mie_latent_spans(mie_index_t cu_seqlens, mie_index_t kv_lens, int32_t requests, int64_t window,
+                     int32_t span_table_width, int64_t row_capacity, int64_t token_capacity, int32_t* spans,
+                     int32_t* span_lens, int32_t* span_table, int32_t* status, void* stream);
+int mie_latent_gather(const void* pages, int64_t page_stride, int64_t slot_stride, const int32_t* spans,
+                      mie_index_t kv_lens, mie_index_t block_tables, void* out, int64_t rows, int32_t cols,
+                      int32_t requests, int32_t dtype, int32_t block_size, int32_t num_blocks, int32_t table_width,
+                      int32_t* status, void* stream);
+
+/*
+ * Decode attention whose heads all read one cached row per token, bf16:
+ * the key is the whole row (dim entries), the value its first value_dim.
+ *   out = sum_j exp(s_j) c_j[0 : value_dim] / (exp(sinks[head]) + sum_j exp(s_j)),
+ *   s_j = (q . c_j) * scale over the last `window` tokens (0: all)
+ * pages [num_blocks, 1, block_size, dim]; dim a multiple of 8 up to 640,
+ * value_dim one up to 512.  Work plan as in mie_sink_decode_attention (use_plan
+ * reuses the plan the scratch holds), scratch mie_latent_decode_scratch_bytes.
+ */
+int mie_latent_decode_supported(int32_t dim, int32_t value_dim, int32_t block_size, int32_t dtype);
+int64_t mie_latent_decode_scratch_bytes(int32_t batch, int32_t heads, int32_t value_dim, int64_t max_total_tokens);
+int mie_latent_decode_attention(const void* query, int64_t q_row_stride, int64_t q_head_stride, void* out,
+                                int64_t o_row_stride, int64_t o_head_stride, mie_view4_t pages,
+                                mie_index_t block_tables, mie_index_t sequence_lengths, int32_t batch, int32_t heads,
+                                int32_t dim, int32_t value_dim, int32_t block_size, int32_t num_blocks,
+                                int32_t table_width, int32_t dtype, float scale, int64_t window, const float* sinks,
+                                int32_t split_policy, void* scratch, int64_t scratch_bytes, int32_t use_plan,
+                                int32_t* status, void* stream);
+
+/*
+ * Decayed outer products: per head S <- decay S + k v^T, o = S^T q with
+ * q, k, v = silu of the row [q heads x dim | k heads x dim | v heads x
+ * value_dim]; out [tokens, heads x value_dim] T, sums and state fp32.
+ * Gated average: S <- (1 - z) S + z c with z = sigmoid(first part + z_bias),
+ * u = second part + u_bias, c = u + 1/2 (u >= 0) or sigmoid(u), out = S *
+ * silu(third part), rows of three parts of `width`.
+ *
+ * State: fp32 rows of slot_stride floats, `state` the layer's part of slot 0,
+ * slots[request] the request's row; a sequence whose first token here has
+ * position 0 starts from zero.  cu_seqlens NULL: token t is one step of
+ * request t.  Otherwise request r owns tokens cu_seqlens[r] ... [r + 1] - 1,
+ * cut into segments of segment_tokens (a multiple of 64) that run in parallel
+ * when `carry` holds (tokens / segment_tokens + requests) x (heads x dim x
+ * value_dim, or 2 x width) floats; carry NULL: one segment per request.
+ * mie_outer_recurrence_chunked: whether chunks take the tensor-core form.
+ */
+int mie_outer_recurrence_chunked(int32_t dim, int32_t value_dim, int32_t dtype);
+int mie_outer_recurrence(const void* rows, int64_t ld, const float* decay, void* out, int64_t ldo, float* state,
+                         int64_t slot_stride, int32_t num_slots, mie_index_t slots, mie_index_t positions,
+                         mie_index_t cu_seqlens, int32_t requests, int32_t segment_tokens, float* carry,
+                         int64_t carry_floats, int32_t tokens, int32_t heads, int32_t dim, int32_t value_dim,
+                         int32_t dtype, int32_t* status, void* stream);
+int mie_gated_average(const void* rows, int64_t ld, const void* z_bias, const void* u_bias, void* out, int64_t ldo,
+                      float* state, int64_t slot_stride, int32_t num_slots, mie_index_t slots, mie_index_t positions,
+                      mie_index_t cu_seqlens, int32_t requests, int32_t segment_tokens, float* carry,
+                      int64_t carry_floats, int32_t tokens, int32_t width, int32_t dtype, int32_t* status,
+                      void* stream);
 
 #ifdef __cplusplus
 }

@@ -24,6 +24,7 @@ STATUS_MAX_LENGTH = 32
 STATUS_CAPACITY = 64
 STATUS_NO_TOKEN = 128
 STATUS_BAD_TOKEN = 256
+STATUS_BAD_SLOT = 512
 
 GEMM_NO_WEIGHT_PREFETCH = 1
 
@@ -37,6 +38,7 @@ STATUS_MESSAGES = {
     STATUS_CAPACITY: "decode work plan exceeded its scratch capacity",
     STATUS_NO_TOKEN: "greedy sampling found no candidate for a row (token 0 was substituted)",
     STATUS_BAD_TOKEN: "a token id lies outside the vocabulary",
+    STATUS_BAD_SLOT: "a state slot lies outside the state buffer",
 }
 
 DTYPE_CODES = {torch.bfloat16: 0, torch.float16: 1, torch.float32: 2}
@@ -152,6 +154,36 @@ _SIGNATURES: dict[str, tuple[object, list[object]]] = {
                                                   View4T, IndexT, IndexT, IndexT, c_int32, c_int32, c_int32, c_int32,
                                                   c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_float,
                                                   c_int64, c_void_p, c_void_p, c_void_p]),
+    "mie_residual_norm": (ctypes.c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_float, c_void_p, c_void_p,
+                                         c_int64, c_int32, c_int32, c_int32, c_float, c_void_p]),
+    "mie_gelu": (ctypes.c_int, [c_void_p, c_int64, IndexT, c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int32,
+                                c_int32, c_int32, c_void_p, c_void_p]),
+    "mie_gated_norm": (ctypes.c_int, [c_void_p, c_int64, c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_int32,
+                                      c_int32, c_int32, c_float, c_void_p]),
+    "mie_softcap": (ctypes.c_int, [c_void_p, c_int64, c_float, c_void_p]),
+    "mie_latent_norm_write": (ctypes.c_int, [c_void_p, c_int64, c_int32, c_int32, c_int32, c_int32, c_void_p,
+                                             c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64, c_int64,
+                                             IndexT, IndexT, IndexT, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                             c_int32, c_float, c_void_p, c_void_p]),
+    "mie_rotate_heads": (ctypes.c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, IndexT, c_void_p,
+                                        c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p]),
+    "mie_latent_spans": (ctypes.c_int, [IndexT, IndexT, c_int32, c_int64, c_int32, c_int64, c_int64, c_void_p,
+                                        c_void_p, c_void_p, c_void_p, c_void_p]),
+    "mie_latent_gather": (ctypes.c_int, [c_void_p, c_int64, c_int64, c_void_p, IndexT, IndexT, c_void_p, c_int64,
+                                         c_int32, c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
+    "mie_latent_decode_supported": (ctypes.c_int, [c_int32, c_int32, c_int32, c_int32]),
+    "mie_latent_decode_scratch_bytes": (c_int64, [c_int32, c_int32, c_int32, c_int64]),
+    "mie_latent_decode_attention": (ctypes.c_int, [c_void_p, c_int64, c_int64, c_void_p, c_int64, c_int64, View4T,
+                                                   IndexT, IndexT, c_int32, c_int32, c_int32, c_int32, c_int32,
+                                                   c_int32, c_int32, c_int32, c_float, c_int64, c_void_p, c_int32,
+                                                   c_void_p, c_int64, c_int32, c_void_p, c_void_p]),
+    "mie_outer_recurrence_chunked": (ctypes.c_int, [c_int32, c_int32, c_int32]),
+    "mie_outer_recurrence": (ctypes.c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_int64, c_void_p, c_int64,
+                                            c_int32, IndexT, IndexT, IndexT, c_int32, c_int32, c_void_p, c_int64,
+                                            c_int32, c_int32, c_int32, c_int32, c_int32, c_void_p, c_void_p]),
+    "mie_gated_average": (ctypes.c_int, [c_void_p, c_int64, c_void_p, c_void_p, c_void_p, c_int64, c_void_p, c_int64,
+                                         c_int32, IndexT, IndexT, IndexT, c_int32, c_int32, c_void_p, c_int64,
+                                         c_int32, c_int32, c_int32, c_void_p, c_void_p]),
 }
 
 _lib: ctypes.CDLL | None = None

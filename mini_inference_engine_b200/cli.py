@@ -58,7 +58,8 @@ def run_generate(args: argparse.Namespace) -> int:
     page = 16
     pages = args.max_batch * (-(-longest // page) + 1)
     runner = load_runner(args.model, dtype=DTYPES[args.dtype], random_seed=args.random_weights, num_pages=pages,
-                         max_batch=args.max_batch, max_context=max(longest, 1024))
+                         max_batch=args.max_batch, max_context=max(longest, 1024),
+                         state_slots=args.max_batch * (2 if args.prefix_cache else 1))
     batcher = ContinuousBatcher(runner, max_prefill_tokens=args.max_prefill_tokens, mixed=args.mixed,
                                 prefix_cache=args.prefix_cache)
     for index, prompt in enumerate(prompts):
@@ -81,7 +82,7 @@ def run_trace(args: argparse.Namespace) -> int:
     page = 16
     pages = -(-max(args.max_tokens, 1) // page) + 256  # every live request may leave one page partly filled
     runner = load_runner(args.model, dtype=DTYPES[args.dtype], num_pages=pages, max_batch=8,
-                         max_context=args.max_tokens + page)
+                         max_context=args.max_tokens + page, state_slots=256)
     session = TraceSession(runner)
     for line in sys.stdin:
         if not line.strip():

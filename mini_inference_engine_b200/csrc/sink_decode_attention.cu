@@ -12,74 +12,6 @@ namespace mie {
 namespace {
 
 constexpr int kMaxBoxes = 4;  // head sizes up to 256
-constexpr int kMergeWarps = 4;
-
-template <typename T, int VH>
-__global__ void __launch_bounds__(kMergeWarps * 32) merge_rows_kernel(DecodeParams p) {
-  __shared__ float part[kMergeWarps][2 + VH * 64];
-  chain_wait();
-  chain_release();
-  const int b = blockIdx.x / p.q_heads, head = blockIdx.x % p.q_heads;
-  const int first = p.sc.offsets[b], n = p.sc.offsets[b + 1] - first;
-  if (n <= 1) return;
-  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  float big = -INFINITY, lsum = 0.f, acc[VH][2];
-#pragma unroll
-  for (int x = 0; x < VH; ++x) acc[x][0] = acc[x][1] = 0.f;
-#pragma unroll 4
-  for (int i = warp; i < n; i += kMergeWarps) {
-    const long long row = ((long long)first + i) * p.q_heads + head;
-    const float mi = p.sc.part_m[row], li = p.sc.part_l[row];
-    const float mn = fmaxf(big, mi);
-    const float wo = exp2f(big - mn), wi = exp2f(mi - mn);
-    lsum = lsum * wo + li * wi;
-    big = mn;
-#pragma unroll
-    for (int x = 0; x < VH; ++x) {
-      const int d = x * 64 + 2 * lane;
-      if (d < p.vdim) {
-        const float2 o = *reinterpret_cast<const float2*>(p.sc.part_o + row * p.vdim + d);
-        acc[x][0] = acc[x][0] * wo + o.x * wi;
-        acc[x][1] = acc[x][1] * wo + o.y * wi;
-      }
-    }
-  }
-  float* mine = part[warp];
-  if (lane == 0) {
-    mine[0] = big;
-    mine[1] = lsum;
-  }
-#pragma unroll
-  for (int x = 0; x < VH; ++x) {
-    mine[2 + x * 64 + 2 * lane] = acc[x][0];
-    mine[2 + x * 64 + 2 * lane + 1] = acc[x][1];
-  }
-  __syncthreads();
-  if (warp != 0) return;
-  big = -INFINITY;
-  for (int w = 0; w < kMergeWarps; ++w) big = fmaxf(big, part[w][0]);
-  lsum = 0.f;
-#pragma unroll
-  for (int x = 0; x < VH; ++x) acc[x][0] = acc[x][1] = 0.f;
-  for (int w = 0; w < kMergeWarps; ++w) {
-    const float mw = part[w][0];
-    if (mw == -INFINITY) continue;  // this warp had no chunk
-    const float wt = exp2f(mw - big);
-    lsum += part[w][1] * wt;
-#pragma unroll
-    for (int x = 0; x < VH; ++x) {
-      acc[x][0] += part[w][2 + x * 64 + 2 * lane] * wt;
-      acc[x][1] += part[w][2 + x * 64 + 2 * lane + 1] * wt;
-    }
-  }
-  const float inv = 1.f / fmaxf(lsum, 1.17549435e-38f);
-  T* orow = reinterpret_cast<T*>(p.out.ptr) + (long long)b * p.out.s[0] + (long long)head * p.out.s[1];
-#pragma unroll
-  for (int x = 0; x < VH; ++x) {
-    const int d = x * 64 + 2 * lane;
-    if (d < p.vdim) *reinterpret_cast<uint32_t*>(orow + d) = Mma16816<T>::pack(acc[x][0] * inv, acc[x][1] * inv);
-  }
-}
 
 template <int KH, int VH>
 int launch_sink(const DecodeParams& p, const CUtensorMap& kmap, const CUtensorMap& vmap, cudaStream_t stream) {

@@ -25,14 +25,17 @@ def sinusoid_turns(width: int, base: float, device: torch.device) -> torch.Tenso
 
 
 def embed_tokens(ids, table, positions, token_to_sequence, block_tables, *, scale: float, page: int, num_pages: int,
-                 bigram=None, mul_prev: int = 0, mul_cur: int = 0, history=None, turns=None,
-                 status: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor]:
-    """``(fp32 rows, activation rows)`` of table[id] * scale (+ bigram row) (+ sinusoid).  ``history``
-    (``[pages, page]`` int32) is the paged record of token ids the bigram part reads a predecessor from."""
+                 bigram=None, mul_prev: int = 0, mul_cur: int = 0, history=None, turns=None, keep_rows: bool = True,
+                 status: torch.Tensor) -> tuple[torch.Tensor, torch.Tensor | None]:
+    """``(fp32 rows, activation rows)`` of table[id] * scale (+ bigram row) (+ sinusoid); without ``keep_rows`` only
+    the fp32 rows.  ``history`` (``[pages, page]`` int32) is the paged record of token ids the bigram part reads a
+    predecessor from."""
 
     tokens, width = int(ids.shape[0]), int(table.shape[1])
     out32 = torch.empty(tokens, width, dtype=torch.float32, device=table.device)
-    out = out32 if table.dtype == torch.float32 else torch.empty(tokens, width, dtype=table.dtype, device=table.device)
+    out = out32 if table.dtype == torch.float32 else None
+    if out is None and keep_rows:
+        out = torch.empty(tokens, width, dtype=table.dtype, device=table.device)
     _lib.check(_lib.load().mie_embed_tokens(
         _lib.index_arg(ids), _lib.ptr(table), int(table.shape[0]), float(scale), _lib.ptr(bigram),
         0 if bigram is None else int(bigram.shape[0]) - 1, int(mul_prev), int(mul_cur), _lib.ptr(turns),
@@ -93,4 +96,52 @@ def clamped_glu(gate_up, *, limit: float, slope: float, up_offset: float) -> tor
     return out
 
 
-__all__ = ["clamped_glu", "embed_tokens", "qkv_norm_mix_write", "sinusoid_turns", "sum_rms_norm"]
+def residual_norm_(x32, y, y_weight, next_weight=None, *, alpha: float, eps: float, keep_rows: bool = True):
+    """``x32 += alpha * rms_norm(y) * y_weight`` in place, then the rows the next product reads, in the weights' dtype:
+    ``rms_norm(x32) * next_weight``, or ``x32`` itself without a next weight.  ``keep_rows=False``: only ``x32``."""
+
+    rows, cols = x32.shape
+    if next_weight is None and y_weight.dtype == torch.float32:
+        out = x32 if keep_rows else None
+        target = None
+    else:
+        out = target = torch.empty(rows, cols, dtype=y_weight.dtype, device=x32.device) if keep_rows else None
+    _lib.check(_lib.load().mie_residual_norm(
+        _lib.ptr(x32), x32.stride(0), _lib.ptr(y), y.stride(0), _lib.ptr(y_weight), float(alpha),
+        _lib.ptr(next_weight), _lib.ptr(target), cols, rows, cols, _lib.DTYPE_CODES[y_weight.dtype], float(eps),
+        _lib.stream_arg(x32.device)))
+    return out
+
+
+def gelu(x, *, ids=None, table=None, status: torch.Tensor | None = None) -> torch.Tensor:
+    """tanh-form gelu of rows, times the rows ``table[ids]`` (a column slice of a wider table) when given."""
+
+    rows, cols = x.shape
+    out = torch.empty(rows, cols, dtype=x.dtype, device=x.device)
+    _lib.check(_lib.load().mie_gelu(
+        _lib.ptr(x), x.stride(0), _lib.index_arg(ids), _lib.ptr(table), 0 if table is None else table.stride(0),
+        0 if table is None else int(table.shape[0]), _lib.ptr(out), cols, rows, cols, _lib.DTYPE_CODES[x.dtype],
+        _lib.ptr(status), _lib.stream_arg(x.device)))
+    return out
+
+
+def gated_rms_norm(x, gate, weight, *, eps: float) -> torch.Tensor:
+    """rms_norm(x) * weight * sigmoid(gate) over whole rows."""
+
+    rows, cols = x.shape
+    out = torch.empty(rows, cols, dtype=x.dtype, device=x.device)
+    _lib.check(_lib.load().mie_gated_norm(
+        _lib.ptr(x), x.stride(0), _lib.ptr(gate), gate.stride(0), _lib.ptr(weight), _lib.ptr(out), cols, rows, cols,
+        _lib.DTYPE_CODES[x.dtype], float(eps), _lib.stream_arg(x.device)))
+    return out
+
+
+def softcap_(logits, cap: float) -> torch.Tensor:
+    """cap * tanh(logits / cap) in place on contiguous fp32 logits."""
+
+    _lib.check(_lib.load().mie_softcap(_lib.ptr(logits), logits.numel(), float(cap), _lib.stream_arg(logits.device)))
+    return logits
+
+
+__all__ = ["clamped_glu", "embed_tokens", "gated_rms_norm", "gelu", "qkv_norm_mix_write", "residual_norm_",
+           "sinusoid_turns", "softcap_", "sum_rms_norm"]

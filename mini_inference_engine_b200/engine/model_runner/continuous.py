@@ -20,6 +20,11 @@ written (the reference switches its decode graphs OFF when prefix reuse is on,
 engine/serving/chunked_prefill.py:126-127; here a shared page is just the same id in two block-table rows, so
 the captured decode and mixed steps run unchanged).  Pages are reference-counted; a prefix page nobody uses
 stays cached until the pool needs it back.
+
+A runner with recurrent layers gives every live request a state slot.  Its prefix cache shares pages only up to a
+page border whose recurrent state has been kept as well: spare slots (those beyond ``max_batch``) hold copies of the
+state at the page borders where prompt chunks ended, least recently used first out, and a request that borrows pages
+starts from a copy of that state.
 """
 
 from __future__ import annotations
@@ -69,6 +74,26 @@ class PagePool:
         self._promised -= unused_promise
 
 
+class SlotPool:
+    """Free list of the state slots of a recurrent runner (``size`` 0: a runner without recurrent state)."""
+
+    def __init__(self, size: int) -> None:
+        self.size = int(size)
+        self._free = list(range(self.size - 1, -1, -1))
+
+    @property
+    def free_slots(self) -> int:
+        return len(self._free)
+
+    def take(self) -> int:
+        if not self._free:
+            raise PagePoolExhausted("no free state slot")
+        return self._free.pop()
+
+    def give_back(self, slot: int) -> None:
+        self._free.append(slot)
+
+
 @dataclass
 class _Request:
     rid: object
@@ -80,6 +105,7 @@ class _Request:
     generated: list[int] = field(default_factory=list)
     borrowed: int = 0          # leading pages taken over from the prefix cache at admission
     published: int = 0         # leading whole prompt pages already offered to the prefix cache
+    slot: int | None = None    # state slot (recurrent runners)
 
     @property
     def decoding(self) -> bool:
@@ -111,6 +137,10 @@ class ContinuousBatcher:
         if self.mixed:
             self.max_prefill_tokens = min(self.max_prefill_tokens, max(runner.chunk_buckets))
         self.pool = PagePool(runner.num_pages)
+        self.slots = SlotPool(getattr(runner, "num_slots", 0))
+        if self.slots.size and self.slots.size < runner.max_batch:
+            raise ValueError("a recurrent runner needs a state slot per request of a full batch")
+        self._prefix_states: OrderedDict[tuple, int] = OrderedDict()  # prefix key -> slot with the state after it
         self.waiting: deque[_Request] = deque()
         self.live: list[_Request] = []   # admission order; decode rows are the decoding ones, in this order
         self.results: dict[object, list[int]] = {}
@@ -146,7 +176,29 @@ class ContinuousBatcher:
             if cached is None:
                 break
             hits.append(cached)
+        while self.slots.size and hits and self._page_key[hits[-1]] not in self._prefix_states:
+            hits.pop()  # the recurrent state at this border is not known
         return hits
+
+    def _drop_prefix_state(self, key: tuple) -> None:
+        slot = self._prefix_states.pop(key, None)
+        if slot is not None:
+            self.slots.give_back(slot)
+
+    def _keep_prefix_state(self, request: _Request) -> None:
+        """Copy the request's recurrent state to a spare slot when its last chunk ended on a page border."""
+
+        page, spare = self.runner.shape.page, self.slots.size - self.runner.max_batch
+        if spare < 1 or request.prefilled % page or request.prefilled > len(request.prompt):
+            return
+        *_, key = self._prefix_keys(request, request.prefilled // page)
+        if key not in self._prefix_pages or key in self._prefix_states:
+            return
+        if len(self._prefix_states) >= spare:
+            self._drop_prefix_state(next(iter(self._prefix_states)))
+        slot = self.slots.take()
+        self.runner.copy_state(request.slot, slot)
+        self._prefix_states[key] = slot
 
     def _evict(self, wanted: int, keep: set[int]) -> None:
         """Hand cached prefix pages nobody uses back to the pool, oldest first, until ``wanted`` can be promised."""
@@ -158,6 +210,7 @@ class ContinuousBatcher:
                 del self._prefix_pages[key]
                 del self._page_key[cached]
                 self._refs.pop(cached, None)
+                self._drop_prefix_state(key)
                 self.pool.give_back([cached], 0)
 
     def _admit(self) -> None:
@@ -179,6 +232,12 @@ class ContinuousBatcher:
             request.borrowed = request.published = len(hits)
             request.prefilled = len(hits) * page
             self.prefix_hits += request.prefilled
+            if self.slots.size:
+                request.slot = self.slots.take()
+                if hits:
+                    key = self._page_key[hits[-1]]
+                    self._prefix_states.move_to_end(key)
+                    self.runner.copy_state(self._prefix_states[key], request.slot)
             self.live.append(self.waiting.popleft())
 
     def _grow(self, request: _Request, tokens: int) -> None:
@@ -215,6 +274,8 @@ class ContinuousBatcher:
                         del self._refs[used]
                         private.append(used)  # cached prefix pages stay out of the free list until evicted
                 self.pool.give_back(private, request.promised)
+                if request.slot is not None:
+                    self.slots.give_back(request.slot)
             else:
                 still.append(request)
         self.live = still  # order kept: rows are compacted, not shuffled
@@ -227,12 +288,15 @@ class ContinuousBatcher:
                 del self._prefix_pages[key]
                 del self._page_key[cached]
                 self._refs.pop(cached, None)
+                self._drop_prefix_state(key)
                 self.pool.give_back([cached], 0)
 
     # -- one iteration ------------------------------------------------------------------------------
 
     def _plan_chunks(self, budget: int) -> list[tuple[_Request, int, int]]:
-        """(request, start, count) for the partial prompts, shortest remaining first, inside the budget."""
+        """(request, start, count) for the partial prompts, shortest remaining first, inside the budget.  A chunk that
+        would run past the last page border a later request can share stops there when that border's recurrent state
+        is to be kept."""
 
         chunks = []
         partial = sorted((r for r in self.live if not r.decoding), key=lambda r: len(r.prompt) - r.prefilled)
@@ -240,6 +304,10 @@ class ContinuousBatcher:
             if budget <= 0 or len(chunks) >= self.runner.max_chunks:
                 break
             count = min(len(request.prompt) - request.prefilled, budget)
+            if self.prefix_cache and self.slots.size:
+                border = (len(request.prompt) - 1) // self.runner.shape.page * self.runner.shape.page
+                if request.prefilled < border < request.prefilled + count:
+                    count = border - request.prefilled
             chunks.append((request, request.prefilled, count))
             budget -= count
         return chunks
@@ -266,9 +334,11 @@ class ContinuousBatcher:
         decode_lengths = [len(r.prompt) + len(r.generated) for r in decoding]
         decode_blocks = [r.pages for r in decoding]
         chunk_items = [(r.prompt[start:start + count], start, r.pages) for r, start, count in chunks]
+        chunking = [r for r, _, _ in chunks]
         if self.mixed and chunks:
             record["kind"] = "mixed"
-            decode_tokens, chunk_tokens = self._mixed(decode_ids, decode_lengths, decode_blocks, chunk_items)
+            decode_tokens, chunk_tokens = self._mixed(decode_ids, decode_lengths, decode_blocks, chunk_items,
+                                                      self._slots_of([*decoding, *chunking]))
         else:
             decode_tokens, chunk_tokens = [], []
             if decoding:
@@ -276,7 +346,7 @@ class ContinuousBatcher:
                 decode_tokens = self._decode(decoding, decode_ids, decode_lengths, decode_blocks, record)
             if chunks:
                 record["kind"] = "decode+prefill" if decoding else "prefill"
-                chunk_tokens = self._prefill(chunk_items)
+                chunk_tokens = self._prefill(chunk_items, self._slots_of(chunking))
         for request, token in zip(decoding, decode_tokens):
             request.generated.append(int(token))
             produced.append((request.rid, int(token)))
@@ -284,6 +354,7 @@ class ContinuousBatcher:
             request.prefilled = start + count
             if self.prefix_cache:
                 self._publish(request)
+                self._keep_prefix_state(request)
             if request.decoding:  # the chunk completed the prompt: its last row gave the first new token
                 request.generated.append(int(token))
                 produced.append((request.rid, int(token)))
@@ -291,22 +362,27 @@ class ContinuousBatcher:
         self._retire()
         return produced
 
+    def _slots_of(self, requests) -> dict:
+        """The keyword with the requests' state slots, for runners that have them."""
+
+        return {"slots": [r.slot for r in requests]} if self.slots.size else {}
+
     def _decode(self, decoding, ids, lengths, blocks, record) -> list[int]:
-        runner = self.runner
+        runner, slots = self.runner, self._slots_of(decoding)
         if self.use_graphs:
-            tokens, h2d, _ = runner.decode_rows([r.rid for r in decoding], ids, lengths, blocks)
+            tokens, h2d, _ = runner.decode_rows([r.rid for r in decoding], ids, lengths, blocks, **slots)
             record["h2d_bytes"] = h2d
             record["bucket"] = next(b for b in runner.decode_buckets if b >= len(decoding))
             return tokens
-        return eager_step(runner, ids, lengths, blocks, []).tolist()
+        return eager_step(runner, ids, lengths, blocks, [], **slots).tolist()
 
-    def _prefill(self, chunk_items) -> list[int]:
-        return eager_step(self.runner, [], [], [], chunk_items).tolist()
+    def _prefill(self, chunk_items, slots) -> list[int]:
+        return eager_step(self.runner, [], [], [], chunk_items, **slots).tolist()
 
-    def _mixed(self, ids, lengths, blocks, chunk_items) -> tuple[list[int], list[int]]:
+    def _mixed(self, ids, lengths, blocks, chunk_items, slots) -> tuple[list[int], list[int]]:
         if self.use_graphs:
-            return self.runner.mixed_rows(ids, lengths, blocks, chunk_items)
-        out, live = eager_step(self.runner, ids, lengths, blocks, chunk_items).tolist(), len(ids)
+            return self.runner.mixed_rows(ids, lengths, blocks, chunk_items, **slots)
+        out, live = eager_step(self.runner, ids, lengths, blocks, chunk_items, **slots).tolist(), len(ids)
         return out[:live], out[live:]
 
     def run(self, max_iterations: int = 100000) -> dict[object, list[int]]:
@@ -322,4 +398,4 @@ class ContinuousBatcher:
         return self.results
 
 
-__all__ = ["ContinuousBatcher", "PagePool", "PagePoolExhausted"]
+__all__ = ["ContinuousBatcher", "PagePool", "PagePoolExhausted", "SlotPool"]

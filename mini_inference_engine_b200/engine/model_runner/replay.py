@@ -12,7 +12,7 @@ from dataclasses import dataclass, field
 
 import torch
 
-from .continuous import PagePool
+from .continuous import PagePool, SlotPool
 from .step_runner import PagedStepRunner, eager_step
 
 
@@ -20,6 +20,7 @@ from .step_runner import PagedStepRunner, eager_step
 class _Sequence:
     pages: list[int] = field(default_factory=list)
     length: int = 0
+    slot: int | None = None
 
 
 @dataclass(frozen=True)
@@ -35,12 +36,16 @@ class TraceSession:
     def __init__(self, runner: PagedStepRunner) -> None:
         self.runner = runner
         self.pool = PagePool(runner.num_pages)
+        self.slots = SlotPool(getattr(runner, "num_slots", 0))
         self.sequences: dict[object, _Sequence] = {}
 
     def _extend(self, rid, count: int) -> _Sequence:
-        sequence = self.sequences.setdefault(rid, _Sequence())
+        sequence = self.sequences.get(rid) or _Sequence()
         if sequence.length + count > self.runner.max_context:
             raise ValueError(f"request {rid!r} grows past max_context {self.runner.max_context}")
+        if self.slots.size and sequence.slot is None:
+            sequence.slot = self.slots.take()
+        self.sequences[rid] = sequence
         while len(sequence.pages) * self.runner.shape.page < sequence.length + count:
             self.pool.promise(1)
             sequence.pages.append(self.pool.take())
@@ -70,7 +75,9 @@ class TraceSession:
         wanted = [starts[e.rid] + place for e in active for place in e.want]
         out = eager_step(
             self.runner, [e.tokens[0] for e, _ in decode], [s.length + 1 for _, s in decode], [s.pages for _, s in decode],
-            [(e.tokens, s.length, s.pages) for e, s in chunks], logit_rows=wanted or [0], return_logits=True)
+            [(e.tokens, s.length, s.pages) for e, s in chunks],
+            slots=[s.slot for _, s in (*decode, *chunks)] if self.slots.size else (), logit_rows=wanted or [0],
+            return_logits=True)
         for entry, sequence in (*decode, *chunks):
             sequence.length += len(entry.tokens)
         logits = out[1].float().cpu() if wanted else None
@@ -82,6 +89,8 @@ class TraceSession:
             sequence = self.sequences.pop(rid, None)
             if sequence is not None:
                 self.pool.give_back(sequence.pages, 0)
+                if sequence.slot is not None:
+                    self.slots.give_back(sequence.slot)
 
 
 __all__ = ["TraceEntry", "TraceSession"]

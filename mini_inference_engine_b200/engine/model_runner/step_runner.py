@@ -5,6 +5,9 @@ A runner owns a pool of request pages followed by scratch pages, and two forward
 ``PagedStepRunner`` is everything around those two that does not depend on the model: bucket selection, padding
 rows on private scratch pages, capture and replay, packing of host metadata, greedy generation.  A model design
 subclasses it with its weights, its cache tensors and the two forwards; ``ContinuousBatcher`` drives any of them.
+
+A design with recurrent layers also keeps a state slot per request: every row of a step then carries the slot of its
+request next to its block-table row, and padding rows have private scratch slots.
 """
 
 from __future__ import annotations
@@ -45,7 +48,8 @@ class DecodeBuffers:
 
     Rows ``[0, live)`` carry requests, the rest are padding rows: token 0, length 1 and a one-entry table
     pointing at the row's OWN scratch page, so a padding row writes and reads offset 0 of a page no request
-    and no other padding row uses.  ``scratch_pages`` must hold ``batch`` distinct page ids.
+    and no other padding row uses.  ``scratch_pages`` must hold ``batch`` distinct page ids.  With ``scratch_slots``
+    (as many distinct state slots) the rows carry state slots too.
 
     Host side.  Ids and lengths (12 bytes a row) are copied whole every step.  The block tables are not:
     a pinned host mirror remembers, per row, who owns it and how many table entries the device already
@@ -56,7 +60,7 @@ class DecodeBuffers:
     """
 
     def __init__(self, batch: int, table_width: int, device: torch.device, scratch_pages=None,
-                 page: int = 16) -> None:
+                 page: int = 16, scratch_slots=None) -> None:
         self.batch, self.table_width, self.page = batch, table_width, page
         self.advance = False  # True when the captured graph feeds its tokens back and bumps the lengths
         self.scratch_pages = None if scratch_pages is None else tuple(int(p) for p in scratch_pages[:batch])
@@ -79,6 +83,11 @@ class DecodeBuffers:
         self.host_lengths = host((batch,), torch.int32, 1)
         self.host_tables = host((batch, table_width), torch.int32, -1)
         self.host_tokens = host((batch,), torch.int64, 0)
+        self.state_slots = self.host_slots = None
+        if scratch_slots is not None:
+            self.scratch_slots = torch.tensor([int(n) for n in scratch_slots[:batch]], dtype=torch.int32)
+            self.state_slots = self.scratch_slots.to(device)
+            self.host_slots = host((batch,), torch.int32, 0)
         self._owners: list[object] = [None] * batch  # None: the device row is in an unknown state
         self._held: list[int] = [0] * batch          # table entries of the row that the device holds
         self.table_bytes_copied = 0                  # running total, for the measurement of the host step
@@ -100,14 +109,16 @@ class DecodeBuffers:
             self._owners = [None] * self.batch
         return copied
 
-    def pack_rows(self, owners, ids, lengths, block_rows) -> int:
+    def pack_rows(self, owners, ids, lengths, block_rows, slots=None) -> int:
         """One step's rows: ``owners[i]`` (any hashable identity of the request in row i), its input token,
-        its length INCLUDING the new token and its page ids.  Rows beyond ``len(owners)`` become padding.
-        Only table entries that changed since the previous call are copied.  Returns the bytes copied."""
+        its length INCLUDING the new token, its page ids and (``slots``) its state slot.  Rows beyond
+        ``len(owners)`` become padding.  Only table entries that changed since the previous call are copied.  Returns the bytes copied."""
 
         live = len(owners)
         if not (len(ids) == len(lengths) == len(block_rows) == live) or live > self.batch:
             raise ValueError("real row counts must agree and fit the graph bucket")
+        if self.host_slots is not None and live and (slots is None or len(slots) != live):
+            raise ValueError("every row of a recurrent model needs a state slot")
         if self.scratch_pages is None and live < self.batch:
             raise ValueError("padding rows need scratch pages")
         page, width = self.page, self.table_width
@@ -150,6 +161,12 @@ class DecodeBuffers:
         self.input_ids.copy_(self.host_ids, non_blocking=True)
         self.sequence_lengths.copy_(self.host_lengths, non_blocking=True)
         copied = self.batch * 12
+        if self.host_slots is not None:
+            if live:
+                self.host_slots[:live] = torch.as_tensor(slots, dtype=torch.int32)
+            self.host_slots[live:] = self.scratch_slots[live:]
+            self.state_slots.copy_(self.host_slots, non_blocking=True)
+            copied += self.batch * 4
         entries = sum(end - first for _, first, end in dirty)
         if len(dirty) > 32 or entries * 4 > self.host_tables.numel():
             self.block_tables.copy_(self.host_tables, non_blocking=True)
@@ -169,10 +186,12 @@ class MixedBuffers:
 
     Table rows ``[0, decode)`` belong to the decode rows, rows ``[decode, decode + chunks)`` to the prompt
     chunks, the last row to the padding "request" that owns every unused chunk token (its pages are scratch).
+    With ``decode_slots`` and ``chunk_slot`` (scratch) every row carries a state slot.
     """
 
     def __init__(self, decode: int, chunk: int, chunks: int, table_width: int, device: torch.device,
-                 decode_scratch: tuple[int, ...], chunk_scratch: tuple[int, ...], page: int) -> None:
+                 decode_scratch: tuple[int, ...], chunk_scratch: tuple[int, ...], page: int,
+                 decode_slots: tuple[int, ...] | None = None, chunk_slot: int = 0) -> None:
         self.decode, self.chunk, self.chunks, self.table_width, self.page = decode, chunk, chunks, table_width, page
         pad_pages = -(-chunk // page)  # pages the padding tokens of this bucket can spread over
         if len(decode_scratch) < decode or len(chunk_scratch) < pad_pages:
@@ -196,21 +215,28 @@ class MixedBuffers:
         self.cu_seqlens, self.host_cu = pair((chunks + 2,), torch.int32)
         self.kv_lens, self.host_kv = pair((chunks + 1,), torch.int32)
         self.logit_rows, self.host_logit_rows = pair((decode + chunks,), torch.int64)
+        self.state_slots = self.host_slots = None
+        if decode_slots is not None:
+            self.scratch_slots = torch.tensor([*decode_slots[:decode], *[chunk_slot] * (chunks + 1)], dtype=torch.int32)
+            self.state_slots, self.host_slots = pair((rows,), torch.int32)
         self.output_tokens = torch.zeros(decode + chunks, dtype=torch.int64, device=device)
         self.host_tokens = torch.zeros(decode + chunks, dtype=torch.int64)
         if pin:
             self.host_tokens = self.host_tokens.pin_memory()
         self.pack([], [], [], [])
 
-    def pack(self, decode_ids, decode_lengths, decode_blocks, chunks) -> int:
+    def pack(self, decode_ids, decode_lengths, decode_blocks, chunks, slots=()) -> int:
         """``decode_*``: the live decode rows (token, length including it, page ids).  ``chunks``: a list of
         ``(token ids, start position, page ids)`` with at most ``self.chunks`` entries and ``self.chunk``
-        tokens in total.  Everything else becomes padding.  Returns the bytes copied to the device."""
+        tokens in total.  ``slots``: state slots of the decode rows and then the chunks.  Everything else becomes
+        padding.  Returns the bytes copied to the device."""
 
         live, page = len(decode_ids), self.page
         total = sum(len(c[0]) for c in chunks)
         if live > self.decode or len(chunks) > self.chunks or total > self.chunk:
             raise ValueError("the step does not fit this mixed bucket")
+        if self.host_slots is not None and len(slots) != live + len(chunks):
+            raise ValueError("every row of a recurrent model needs a state slot")
         ids, seq, pos = self.host_ids, self.host_tok2seq, self.host_tokpos
         tables, lengths = self.host_tables, self.host_lengths
         tables.fill_(-1)
@@ -253,6 +279,12 @@ class MixedBuffers:
         self.host_cu[self.chunks + 1] = self.tokens - self.decode
         self.host_logit_rows[:self.decode] = torch.arange(self.decode, dtype=torch.int64)
         copied = 0
+        if self.host_slots is not None:
+            self.host_slots.copy_(self.scratch_slots)
+            for row, slot in enumerate(slots):
+                self.host_slots[row if row < live else self.decode + row - live] = int(slot)
+            self.state_slots.copy_(self.host_slots, non_blocking=True)
+            copied += self.host_slots.numel() * 4
         for device_tensor, host_tensor in ((self.input_ids, ids), (self.token_to_sequence, seq),
                                            (self.token_positions, pos), (self.block_tables, tables),
                                            (self.decode_lengths, lengths), (self.cu_seqlens, self.host_cu),
@@ -262,15 +294,20 @@ class MixedBuffers:
         return copied
 
 
-def eager_step(runner, decode_ids, decode_lengths, decode_blocks, chunks, *, logit_rows=None,
+def eager_step(runner, decode_ids, decode_lengths, decode_blocks, chunks, *, slots=(), logit_rows=None,
                return_logits: bool = False):
     """One step of a runner from host data without a graph.  ``decode_*``: one token per row (id, length
-    including it, page ids); ``chunks``: ``(token ids, start position, page ids)``.  The flat stream is the
-    decode rows followed by the chunks; ``logit_rows`` picks rows of it (default: every decode row and each
-    chunk's last row).  Returns what the forward returns for those rows."""
+    including it, page ids); ``chunks``: ``(token ids, start position, page ids)``; ``slots``: state slots of the
+    decode rows and then the chunks (recurrent runners).  The flat stream is the decode rows followed by the
+    chunks; ``logit_rows`` picks rows of it (default: every decode row and each chunk's last row).  Returns what
+    the forward returns for those rows."""
 
     device, live = runner.device, len(decode_ids)
     extra = {"return_logits": True} if return_logits else {}
+    if getattr(runner, "recurrent", False):
+        if len(slots) != live + len(chunks):
+            raise ValueError("every row of a recurrent model needs a state slot")
+        extra["state_slots"] = torch.tensor(list(slots), dtype=torch.int32).to(device)
     counts = [len(tokens) for tokens, _, _ in chunks]
     tables = torch.full((live + len(chunks), runner.table_width), -1, dtype=torch.int32)
     for row, pages in enumerate([*decode_blocks, *(pages for _, _, pages in chunks)]):
@@ -290,6 +327,8 @@ def eager_step(runner, decode_ids, decode_lengths, decode_blocks, chunks, *, log
         cu[1:] = torch.tensor(counts, dtype=torch.int32).cumsum(0)
     kv_lens = torch.tensor([start + n for (_, start, _), n in zip(chunks, counts)], dtype=torch.int32).to(device)
     longest = max(counts, default=0)
+    if getattr(runner, "wants_chunk_starts", False):
+        extra["chunk_starts"] = [start for _, start, _ in chunks]
     if not live and logit_rows is None:
         return runner.prefill_forward(flat, tok2seq, tokpos, tables, cu.to(device), kv_lens, longest, **extra)
     if logit_rows is None:
@@ -308,14 +347,17 @@ class PagedStepRunner:
     The pool holds ``num_pages`` request pages followed by scratch pages that only padding rows of a captured
     bucket touch (reference: engine/serving/chunked_prefill.py:133-148 - the extra pages are exclusively scratch,
     the request capacity is unchanged): one page per row of the largest decode bucket and enough pages for the
-    padding tokens of the largest prompt-chunk bucket.
+    padding tokens of the largest prompt-chunk bucket.  ``state_slots`` (recurrent designs) is the number of
+    requests that can hold a state slot; scratch slots for padding rows follow them in the same way.
 
     Subclasses provide ``shape`` (with ``page``, the tokens per page), ``decode_forward`` and ``mixed_forward``.
     """
 
+    wants_chunk_starts = False  # whether the mixed forward takes the chunks' start positions as host numbers
+
     def __init__(self, shape, device: torch.device, *, num_pages: int, max_batch: int, max_context: int,
                  decode_buckets: tuple[int, ...] | None = None, chunk_buckets: tuple[int, ...] = (128, 512),
-                 max_chunks: int = 4) -> None:
+                 max_chunks: int = 4, state_slots: int = 0) -> None:
         self.shape, self.device = shape, device
         self.num_pages, self.max_batch, self.max_context = num_pages, max_batch, max_context
         if decode_buckets is None:
@@ -331,6 +373,11 @@ class PagedStepRunner:
                                                num_pages + self.decode_buckets[-1] + chunk_scratch))
         self.total_pages = num_pages + self.decode_buckets[-1] + chunk_scratch
         self.table_width = -(-max_context // shape.page)
+        self.num_slots = int(state_slots)
+        self.recurrent = self.num_slots > 0
+        self.decode_scratch_slots = tuple(range(self.num_slots, self.num_slots + self.decode_buckets[-1]))
+        self.chunk_scratch_slot = self.num_slots + self.decode_buckets[-1]
+        self.total_slots = self.chunk_scratch_slot + 1 if self.recurrent else 0
         self.status = torch.zeros(1, dtype=torch.int32, device=device)
         # (kind, bucket...) -> (graph, buffers): ("decode", rows, advance) or ("mixed", rows, chunk tokens)
         self._graphs: dict[tuple, tuple[torch.cuda.CUDAGraph, object]] = {}
@@ -374,7 +421,7 @@ class PagedStepRunner:
 
     def prefill_forward(self, input_ids: torch.Tensor, token_to_sequence: torch.Tensor,
                         token_positions: torch.Tensor, block_tables: torch.Tensor, cu_seqlens: torch.Tensor,
-                        kv_lens: torch.Tensor, max_query_len: int, return_logits: bool = False):
+                        kv_lens: torch.Tensor, max_query_len: int, return_logits: bool = False, **extra):
         """Flat ``[tokens]`` forward of packed prompt chunks only (reference: engine/model_runner/qwen3_packed.py:29):
         the mixed forward without decode rows; each request's last row is projected to logits.
         Returns the greedy next token of every request ``[requests]``."""
@@ -382,7 +429,8 @@ class PagedStepRunner:
         last_rows = (cu_seqlens[1:].long() - 1).clamp_min(0)
         return self.mixed_forward(input_ids, token_to_sequence, token_positions, block_tables, decode_rows=0,
                                   decode_lengths=None, cu_seqlens=cu_seqlens, kv_lens=kv_lens,
-                                  max_query_len=max_query_len, logit_rows=last_rows, return_logits=return_logits)
+                                  max_query_len=max_query_len, logit_rows=last_rows, return_logits=return_logits,
+                                  **extra)
 
     def generate(self, prompts: list[list[int]], max_new_tokens: int, *, use_graph: bool = True) -> list[list[int]]:
         """Greedy generation for requests that arrive together: one packed
@@ -398,6 +446,11 @@ class PagedStepRunner:
             raise ValueError("the KV pool is too small for these requests")
         if max(n + max_new_tokens for n in lengths) > self.max_context:
             raise ValueError("a request is longer than max_context")
+        if self.recurrent and batch > self.num_slots:
+            raise ValueError("more requests than state slots")
+        slots = torch.arange(batch, dtype=torch.int32, device=device) if self.recurrent else None
+        extra = {"state_slots": slots} if self.recurrent else {}
+        starts = {"chunk_starts": [0] * batch} if self.wants_chunk_starts else {}
         width = self.table_width
         tables = torch.full((batch, width), -1, dtype=torch.int32)
         cursor = 0
@@ -416,7 +469,8 @@ class PagedStepRunner:
         if bucket is not None:
             # A serving engine captures its buckets once at start-up; capture only touches scratch pages.
             buffers = self.capture(bucket, advance=True)
-        next_ids = self.prefill_forward(flat, tok2seq, tokpos, tables_dev, cu.to(device), kv_lens, max(lengths))
+        next_ids = self.prefill_forward(flat, tok2seq, tokpos, tables_dev, cu.to(device), kv_lens, max(lengths),
+                                        **extra, **starts)
         outputs = [[int(t)] for t in next_ids.tolist()]
         current = kv_lens.clone()
         if buffers is not None:
@@ -427,7 +481,8 @@ class PagedStepRunner:
             self._generation += 1
             buffers.pack_rows([(self._generation, row) for row in range(batch)], [0] * batch,
                               [n + 1 for n in lengths],
-                              [tables[row, :needed[row]].tolist() for row in range(batch)])
+                              [tables[row, :needed[row]].tolist() for row in range(batch)],
+                              list(range(batch)) if self.recurrent else None)
             buffers.input_ids[:batch].copy_(next_ids)
             history = torch.empty(max_new_tokens - 1, batch, dtype=torch.int64, device=device)
             for step in range(max_new_tokens - 1):
@@ -441,7 +496,7 @@ class PagedStepRunner:
         else:
             for _ in range(max_new_tokens - 1):
                 current = current + 1
-                next_ids = self.decode_forward(next_ids, current, tables_dev)
+                next_ids = self.decode_forward(next_ids, current, tables_dev, **extra)
                 for row, token in enumerate(next_ids.tolist()):
                     outputs[row].append(int(token))
         self.check_status()
@@ -461,10 +516,11 @@ class PagedStepRunner:
         if batch > len(self.decode_scratch_pages):
             raise ValueError(f"bucket {batch} exceeds the largest decode bucket {len(self.decode_scratch_pages)}")
         buffers = DecodeBuffers(batch, table_width or self.table_width, self.device, self.decode_scratch_pages,
-                                self.shape.page)
+                                self.shape.page, self.decode_scratch_slots if self.recurrent else None)
         buffers.advance = advance
+        extra = {"state_slots": buffers.state_slots} if self.recurrent else {}
         self._capture(key, buffers, lambda: self.decode_forward(buffers.input_ids, buffers.sequence_lengths,
-                                                                buffers.block_tables), advance)
+                                                                buffers.block_tables, **extra), advance)
         return buffers
 
     def capture_mixed(self, decode: int, chunk: int) -> MixedBuffers:
@@ -474,14 +530,16 @@ class PagedStepRunner:
         if key in self._graphs:
             return self._graphs[key][1]
         buffers = MixedBuffers(decode, chunk, self.max_chunks, self.table_width, self.device,
-                               self.decode_scratch_pages, self.chunk_scratch_pages, self.shape.page)
+                               self.decode_scratch_pages, self.chunk_scratch_pages, self.shape.page,
+                               self.decode_scratch_slots if self.recurrent else None, self.chunk_scratch_slot)
+        extra = {"state_slots": buffers.state_slots} if self.recurrent else {}
 
         def forward():
             return self.mixed_forward(buffers.input_ids, buffers.token_to_sequence, buffers.token_positions,
                                       buffers.block_tables, decode_rows=decode,
                                       decode_lengths=buffers.decode_lengths if decode else None,
                                       cu_seqlens=buffers.cu_seqlens, kv_lens=buffers.kv_lens, max_query_len=chunk,
-                                      logit_rows=buffers.logit_rows)
+                                      logit_rows=buffers.logit_rows, **extra)
 
         self._capture(key, buffers, forward, False)
         return buffers
@@ -517,7 +575,7 @@ class PagedStepRunner:
         torch.cuda.current_stream(self.device).synchronize()
         return buffers.host_tokens, h2d, buffers.host_tokens.numel() * 8
 
-    def decode_rows(self, owners, ids, lengths, block_rows) -> tuple[list[int], int, int]:
+    def decode_rows(self, owners, ids, lengths, block_rows, slots=None) -> tuple[list[int], int, int]:
         """One decode step for the live rows of a continuous batch: the smallest bucket that holds them is
         captured on first use, the rows are packed (padding rows reset, block tables updated incrementally),
         the bucket's graph is replayed and the live rows' tokens are read back (reference:
@@ -528,13 +586,13 @@ class PagedStepRunner:
         if bucket is None:
             raise ValueError(f"{live} rows exceed the largest decode bucket {self.decode_buckets[-1]}")
         buffers = self.capture(bucket)
-        h2d = buffers.pack_rows(owners, ids, lengths, block_rows)
+        h2d = buffers.pack_rows(owners, ids, lengths, block_rows, slots)
         self._graphs[("decode", bucket, False)][0].replay()
         buffers.host_tokens[:live].copy_(buffers.output_tokens[:live], non_blocking=True)
         torch.cuda.current_stream(self.device).synchronize()
         return buffers.host_tokens[:live].tolist(), h2d, live * 8
 
-    def mixed_rows(self, decode_ids, decode_lengths, decode_blocks, chunks) -> tuple[list[int], list[int]]:
+    def mixed_rows(self, decode_ids, decode_lengths, decode_blocks, chunks, slots=()) -> tuple[list[int], list[int]]:
         """One captured mixed step (see ``MixedBuffers.pack``).  Returns the decode rows' tokens and, per
         chunk, the greedy token after its last row (meaningful when the chunk completes its prompt)."""
 
@@ -544,7 +602,7 @@ class PagedStepRunner:
         if decode is None or chunk is None or len(chunks) > self.max_chunks:
             raise ValueError("the step exceeds the largest mixed bucket")
         buffers = self.capture_mixed(decode, chunk)
-        buffers.pack(decode_ids, decode_lengths, decode_blocks, chunks)
+        buffers.pack(decode_ids, decode_lengths, decode_blocks, chunks, slots)
         self._graphs[("mixed", decode, chunk)][0].replay()
         buffers.host_tokens.copy_(buffers.output_tokens, non_blocking=True)
         torch.cuda.current_stream(self.device).synchronize()

@@ -15,6 +15,7 @@ import torch
 
 from .checkpoint import Checkpoint, CheckpointError, load_config
 from .model_runner.qwen3_decode import Qwen3DecodeRunner, Qwen3Shape, Qwen3Weights
+from .model_runner.ripesun import RipesunRunner, RipesunShape, RipesunWeights
 from .model_runner.step_runner import PagedStepRunner
 from .model_runner.tidelorn import TidelornRunner, TidelornShape, TidelornWeights
 
@@ -33,6 +34,7 @@ class ModelDesign:
     checkpoint_weights: Callable                     # (shape, Checkpoint, device, dtype) -> weights
     random_weights: Callable                         # (shape, device, dtype, seed) -> weights
     runner: Callable[..., PagedStepRunner]           # (weights, num_pages=, max_batch=, max_context=, ...) -> runner
+    recurrent: bool = False                          # requests hold a state slot; the runner takes state_slots=
 
 
 DESIGNS: dict[str, ModelDesign] = {}
@@ -56,9 +58,10 @@ def design_for(config: dict) -> ModelDesign:
 
 
 def load_runner(folder: str | Path, *, dtype: torch.dtype = torch.bfloat16, device: torch.device | None = None,
-                random_seed: int | None = None, **runner_options) -> PagedStepRunner:
+                random_seed: int | None = None, state_slots: int | None = None, **runner_options) -> PagedStepRunner:
     """Runner of the model in ``folder``: its checkpoint's weights, or seeded random ones of its configuration
-    when ``random_seed`` is given.  ``runner_options``: ``num_pages``, ``max_batch``, ``max_context`` and so on."""
+    when ``random_seed`` is given.  ``state_slots`` goes to designs with recurrent state, ``runner_options``
+    (``num_pages``, ``max_batch``, ``max_context`` and so on) to every runner."""
 
     config = load_config(folder)
     design = design_for(config)
@@ -70,6 +73,8 @@ def load_runner(folder: str | Path, *, dtype: torch.dtype = torch.bfloat16, devi
         weights = design.checkpoint_weights(shape, Checkpoint(folder), device, dtype)
     else:
         weights = design.random_weights(shape, device, dtype, random_seed)
+    if design.recurrent and state_slots is not None:
+        runner_options["state_slots"] = state_slots
     return design.runner(weights, **runner_options)
 
 
@@ -98,6 +103,12 @@ register(ModelDesign(
     checkpoint_weights=lambda shape, checkpoint, device, dtype: TidelornWeights(shape, checkpoint.take, device, dtype),
     random_weights=lambda shape, device, dtype, seed: TidelornWeights.random(shape, device, seed=seed, dtype=dtype),
     runner=TidelornRunner))
+
+register(ModelDesign(
+    name="Ripesun", dtypes=(torch.bfloat16, torch.float32), shape=RipesunShape.from_config,
+    checkpoint_weights=lambda shape, checkpoint, device, dtype: RipesunWeights(shape, checkpoint.take, device, dtype),
+    random_weights=lambda shape, device, dtype, seed: RipesunWeights.random(shape, device, seed=seed, dtype=dtype),
+    runner=RipesunRunner, recurrent=True))
 
 
 __all__ = ["DESIGNS", "DTYPES", "ModelDesign", "UnsupportedDtype", "design_for", "load_runner", "register"]
