@@ -47,9 +47,10 @@ def parse_args() -> argparse.Namespace:
     parser.add_argument("--layers", type=int, default=None, help="debug: fewer layers (invalid as a result)")
     parser.add_argument("--no-cpu-baseline", action="store_true")
     parser.add_argument("--no-e2e", action="store_true")
-    parser.add_argument("--workload", default="config4", choices=["config4", "config3", "tidelorn"],
+    parser.add_argument("--workload", default="config4", choices=["config4", "config3", "tidelorn", "ripesun"],
                         help="config4: ragged decode sweep point (the headline); config3: 8 x (2048 prompt + 128 new); "
-                             "tidelorn: that design's prefill, decode and kernels beside the Qwen3 runner")
+                             "tidelorn / ripesun: that design's prefill, decode and kernels beside the Qwen3 / Tidelorn "
+                             "runner")
     parser.add_argument("--no-extras", action="store_true",
                         help="skip the extra keys measured after the headline (configs 0-3, FP8 KV cache)")
     parser.add_argument("--breakdown", action="store_true",
@@ -300,19 +301,21 @@ def run_config3(args, shape, device, rank, world, group) -> None:
         leave_together(runner, device)
 
 
-def run_tidelorn(args, device, rank) -> None:
-    """Not the headline: prefill and decode of the Tidelorn design at layer sizes of real models, beside the
-    Qwen3 runner at equal sizes, with every kernel of both against its roofline."""
+def run_design(name: str, device, rank) -> None:
+    """Not the headline: prefill and decode of another design at layer sizes of real models, beside the closest
+    runner at equal sizes, with every kernel of both against its roofline."""
 
     import modelbench
 
+    run, dtype = {"tidelorn": (modelbench.run, "bf16 (Qwen3 arm: fp8_e4m3 GEMM)"),
+                  "ripesun": (modelbench.run_ripesun, "bf16")}[name]
     sampler = ClockSampler(device.index or 0)
     sampler.start()
-    result = modelbench.run(device, measured_peaks()[0], measured_tensor_peak())
+    result = run(device, measured_peaks()[0], measured_tensor_peak())
     clocks = sampler.stop()
     if rank == 0:
-        emit({"workload": "tidelorn", "n_gpus": 1, "data": "synthetic", "dtype": "bf16 (Qwen3 arm: fp8_e4m3 GEMM)",
-              "peaks": measured_peaks()[1], "clocks": clocks, **result})
+        emit({"workload": name, "n_gpus": 1, "data": "synthetic", "dtype": dtype, "peaks": measured_peaks()[1],
+              "clocks": clocks, **result})
 
 
 def run_breakdown(runner, buffers, steps: int, device, rank: int, world: int, concurrency: int) -> None:
@@ -564,8 +567,8 @@ def main() -> None:
         return float(t.item())
 
     shape = Qwen3Shape()
-    if args.workload == "tidelorn":
-        run_tidelorn(args, device, rank)
+    if args.workload in ("tidelorn", "ripesun"):
+        run_design(args.workload, device, rank)
         return
     if args.workload == "config3":
         run_config3(args, shape, device, rank, world, group)

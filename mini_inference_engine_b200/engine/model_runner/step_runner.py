@@ -86,7 +86,7 @@ class DecodeBuffers:
         self.state_slots = self.host_slots = None
         if scratch_slots is not None:
             self.scratch_slots = torch.tensor([int(n) for n in scratch_slots[:batch]], dtype=torch.int32)
-            self.state_slots = self.scratch_slots.to(device)
+            self.state_slots = self.scratch_slots.clone().to(device)
             self.host_slots = host((batch,), torch.int32, 0)
         self._owners: list[object] = [None] * batch  # None: the device row is in an unknown state
         self._held: list[int] = [0] * batch          # table entries of the row that the device holds
