@@ -5,7 +5,8 @@
 // One persistent CTA per SM walks (request, chunk, group of heads) items of the shared split-KV plan in a fixed
 // order: a producer warp streams 16-token slabs of the request's pages into a ring of 64-token stages with TMA
 // (128-byte swizzle, no multicast) and runs ahead across items; eight warps compute on a stage together:
-//   S = Q K^T    warp = (16 heads, 8 * MT keys), whole key size            -> row maxima meet in shared memory
+//   S = Q K^T    warp = (16 heads, 16 * MT keys, every other 16 dims); with one 16-head tile Q stays in registers.  The
+//                pair that shares keys swaps halves of its sums               -> row maxima meet in shared memory
 //   P            exp2 against the common running maximum, as a rounded bf16 part plus its remainder, to shared memory
 //   O += P V     warp = one 64-dim box of the values, all heads, V read transposed from the same stage
 // Scores, weights, sums and O are fp32.  The sink opens the running maximum and the denominator of a request's first
@@ -42,16 +43,17 @@ struct LatentParams {
   int* status;
 };
 
-// Shared memory: K ring | Q | P (rounded, remainder) | row maxima | row sums | barriers.
+// Shared memory: K ring | Q | P (rounded, remainder) | swapped sums | row maxima | row sums | barriers.
 struct LatentLayout {
-  int stage, q, p, maxima, sums, bars, total;
+  int stage, q, p, swap, maxima, sums, bars, total;
 };
 __host__ __device__ inline LatentLayout latent_layout(int key_boxes, int mt) {
   LatentLayout l;
   l.stage = key_boxes * kStageTokens * 128;
   l.q = kRing * l.stage;
   l.p = l.q + key_boxes * mt * 16 * 128;
-  l.maxima = l.p + 2 * mt * 16 * 128;
+  l.swap = l.p + 2 * mt * 16 * 128;
+  l.maxima = l.swap + kComputeWarps * 32 * mt * 4 * 4;
   l.sums = l.maxima + mt * 16 * 8 * 4;
   l.bars = l.sums + mt * 16 * 8 * 4;
   l.total = l.bars + 64;
@@ -66,7 +68,8 @@ struct LatentItem {
   long long first_seen, begin, end;  // first visible token, tokens of the chunk
 };
 
-template <int MT>  // 16-head tiles per item
+// MT: 16-head tiles per item.  BOXES: upper limit of the key's 64-dim boxes.
+template <int MT, int BOXES>
 __global__ void __launch_bounds__(kLatentThreads, 1)
     latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentParams p) {
   using T = __nv_bfloat16;
@@ -93,7 +96,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   const long long capacity = (long long)p.table_width * p.block_size;
   auto item_of = [&](int number) {
     LatentItem it;
-    const int pair = number / p.head_groups;
+    const int pair = number / p.head_groups;  // below the plan's pair count, checked by the callers
     it.group = number % p.head_groups;
     it.request = p.sc.item_seq[pair];
     it.chunk = p.sc.item_chunk[pair];
@@ -149,9 +152,14 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   } else {
     // ---------------- compute ----------------
     const int g = lane >> 2, t = lane & 3;
-    constexpr int kKeys = 8 * MT;           // keys per warp in S
+    // S: warp = (16-head tile mt_s, every other 16-dim step from k_half on, 16 * MT keys of pair kp); after the swap it
+    // owns kKeys of them, group kg.
+    constexpr int kKeys = 8 * MT;
     constexpr int kKeyGroups = 64 / kKeys;
-    const int mt_s = warp % MT, kg = warp / MT;
+    constexpr int kSteps = BOXES * 2;  // 16-dim steps of one half
+    constexpr bool kHoldQ = MT == 1;
+    const int mt_s = warp % MT, k_half = warp / MT % 2, kp = warp / (2 * MT);
+    const int kg = 2 * kp + k_half;
     const int value_boxes = (p.vdim + 63) / 64;
     const int k_steps = (p.dim + 15) / 16;
     const uint32_t q_at = smem_u32(smem + at.q), p_at = smem_u32(smem + at.p);
@@ -159,9 +167,8 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
     float* sums = reinterpret_cast<float*>(smem + at.sums);
     const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_sel = (lane >> 4) & 1;
     const int v_row = (lane & 7) + ((lane >> 3) & 1) * 8, v_sel = (lane >> 4) & 1;
-    // K operand: for MT = 2 sixteen keys x 16 dims per load, for MT = 1 eight keys x 32 dims.
-    const int k_row = MT == 2 ? (lane & 7) + ((lane >> 4) & 1) * 8 : (lane & 7);
-    const int k_sel = MT == 2 ? (lane >> 3) & 1 : lane >> 3;
+    const int k_row = (lane & 7) + ((lane >> 4) & 1) * 8, k_sel = (lane >> 3) & 1;  // sixteen keys x 16 dims per load
+    float* swap = reinterpret_cast<float*>(smem + at.swap);
     int fill = 0;
     bool ok = true;
     for (int number = blockIdx.x; number < total_items; number += gridDim.x) {
@@ -193,6 +200,17 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         }
       }
       compute_sync();
+      auto load_q = [&](int ks, uint32_t (&a)[4]) {
+        ldmatrix_x4(a[0], a[1], a[2], a[3],
+                    q_at + (ks >> 2) * (MT * 16 * 128) + (mt_s * 16 + a_row) * 128 +
+                        ((((ks & 3) * 2 + a_sel) ^ (a_row & 7)) << 4));
+      };
+      uint32_t held[kHoldQ ? kSteps : 1][4];
+      if (kHoldQ) {
+#pragma unroll
+        for (int i = 0; i < kSteps; ++i)
+          if (2 * i + k_half < k_steps) load_q(2 * i + k_half, held[kHoldQ ? i : 0]);
+      }
       for (long long tok0 = it.begin; tok0 < it.end; tok0 += kStageTokens, ++fill) {
         const int s = fill % kRing;
         const bool arrived = ok && mbar_wait_bounded(&full[s], (fill / kRing) & 1u);
@@ -209,40 +227,48 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
           fence_proxy_async_smem();
           compute_sync();
         }
-        // S for (16 heads) x (kKeys keys), two accumulator sets.
-        float sa[2][MT][4];
+        // Half sums of S for 16 heads x 16 * MT keys.
+        float part[2 * MT][4];
 #pragma unroll
-        for (int i = 0; i < 2; ++i)
+        for (int n = 0; n < 2 * MT; ++n) part[n][0] = part[n][1] = part[n][2] = part[n][3] = 0.f;
 #pragma unroll
-          for (int n = 0; n < MT; ++n) sa[i][n][0] = sa[i][n][1] = sa[i][n][2] = sa[i][n][3] = 0.f;
-        const int key_row = kg * kKeys + k_row;
-        const uint32_t k_base = stage + (key_row >> 3) * tok_group + (key_row & 7) * 128;
-        const uint32_t q_base = q_at + (mt_s * 16 + a_row) * 128;
-        auto q_frag = [&](int ks, uint32_t (&a)[4]) {
-          ldmatrix_x4(a[0], a[1], a[2], a[3],
-                      q_base + (ks >> 2) * (MT * 16 * 128) + ((((ks & 3) * 2 + a_sel) ^ (a_row & 7)) << 4));
-        };
-        // Two steps of 16 dims at a time, one accumulator set each; a box holds four steps, so the second is always
-        // inside it (zeros past the end).
-#pragma unroll 2
-        for (int ks = 0; ks < k_steps; ks += 2) {
-          uint32_t a[4], b[4], r[2][4];
-          q_frag(ks, a);
-          q_frag(ks + 1, b);
+        for (int i = 0; i < kSteps; ++i) {
+          const int ks = 2 * i + k_half;
+          if (ks < k_steps) {
+            uint32_t(&q)[4] = held[kHoldQ ? i : 0];
+            if (!kHoldQ) load_q(ks, q);
 #pragma unroll
-          for (int step = 0; step < MT; ++step)
-            ldmatrix_x4(r[step][0], r[step][1], r[step][2], r[step][3],
-                        k_base + (ks >> 2) * dim_group + (((((ks & 3) + step) * 2 + k_sel) ^ (key_row & 7)) << 4));
-          if (MT == 1) {
-            Mma::run(sa[0][0], a[0], a[1], a[2], a[3], r[0][0], r[0][1]);
-            Mma::run(sa[1][0], b[0], b[1], b[2], b[3], r[0][2], r[0][3]);
-          } else {
-#pragma unroll
-            for (int n = 0; n < MT; ++n) {
-              Mma::run(sa[0][n], a[0], a[1], a[2], a[3], r[0][2 * n], r[0][2 * n + 1]);
-              Mma::run(sa[1][n], b[0], b[1], b[2], b[3], r[MT - 1][2 * n], r[MT - 1][2 * n + 1]);
+            for (int np = 0; np < MT; ++np) {
+              const int key_row = (kp * MT + np) * 16 + k_row;
+              uint32_t r0, r1, r2, r3;
+              ldmatrix_x4(r0, r1, r2, r3,
+                          stage + (key_row >> 3) * tok_group + (key_row & 7) * 128 + (ks >> 2) * dim_group +
+                              ((((ks & 3) * 2 + k_sel) ^ (key_row & 7)) << 4));
+              Mma::run(part[2 * np], q[0], q[1], q[2], q[3], r0, r1);
+              Mma::run(part[2 * np + 1], q[0], q[1], q[2], q[3], r2, r3);
             }
           }
+        }
+        // Swap with the warp that has the other dims: each of the pair keeps half of the keys.
+        float sa[MT][4];
+#pragma unroll
+        for (int n = 0; n < MT; ++n) {
+          float4 give;
+          if (k_half == 0) {
+            give = make_float4(part[MT + n][0], part[MT + n][1], part[MT + n][2], part[MT + n][3]);
+            sa[n][0] = part[n][0], sa[n][1] = part[n][1], sa[n][2] = part[n][2], sa[n][3] = part[n][3];
+          } else {
+            give = make_float4(part[n][0], part[n][1], part[n][2], part[n][3]);
+            sa[n][0] = part[MT + n][0], sa[n][1] = part[MT + n][1], sa[n][2] = part[MT + n][2], sa[n][3] = part[MT + n][3];
+          }
+          *reinterpret_cast<float4*>(swap + ((warp * MT + n) * 32 + lane) * 4) = give;
+        }
+        asm volatile("bar.sync %0, 64;" ::"r"(2 + kp * MT + mt_s) : "memory");
+#pragma unroll
+        for (int n = 0; n < MT; ++n) {
+          const int other = k_half == 0 ? warp + MT : warp - MT;
+          const float4 v = *reinterpret_cast<const float4*>(swap + ((other * MT + n) * 32 + lane) * 4);
+          sa[n][0] += v.x, sa[n][1] += v.y, sa[n][2] += v.z, sa[n][3] += v.w;
         }
         float mx[2] = {-INFINITY, -INFINITY};
 #pragma unroll
@@ -250,9 +276,9 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
 #pragma unroll
           for (int e = 0; e < 4; ++e) {
             const int key = kg * kKeys + n * 8 + 2 * t + (e & 1);
-            float v = (sa[0][n][e] + sa[1][n][e]) * p.scale_log2;
+            float v = sa[n][e] * p.scale_log2;
             if (key >= valid || tok0 + key < it.first_seen) v = -INFINITY;
-            sa[0][n][e] = v;
+            sa[n][e] = v;
             mx[e >> 1] = fmaxf(mx[e >> 1], v);
           }
         }
@@ -288,7 +314,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
           const int key = kg * kKeys + n * 8 + 2 * t;
 #pragma unroll
           for (int e = 0; e < 2; ++e) {
-            const float w0 = exp2f(sa[0][n][2 * e] - m_s[e]), w1 = exp2f(sa[0][n][2 * e + 1] - m_s[e]);
+            const float w0 = exp2f(sa[n][2 * e] - m_s[e]), w1 = exp2f(sa[n][2 * e + 1] - m_s[e]);
             l[e] += w0 + w1;
             const int row = mt_s * 16 + g + e * 8;
             uint8_t* dst = smem + at.p + row * 128 + (((key >> 3) ^ (row & 7)) << 4) + (key & 7) * 2;
@@ -385,19 +411,27 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   }
 }
 
-template <int MT>
+template <int MT, int BOXES>
 int launch_latent(const CUtensorMap& map, const LatentParams& p, cudaStream_t stream) {
   const int smem = latent_layout(p.key_boxes, MT).total + 1024;
   static int configured[64] = {0};
   int dev = 0;
   MIE_CUDA(cudaGetDevice(&dev));
   if (dev < 0 || dev >= 64 || configured[dev] < smem) {
-    MIE_CUDA(cudaFuncSetAttribute(latent_decode_kernel<MT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    MIE_CUDA(cudaFuncSetAttribute(latent_decode_kernel<MT, BOXES>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     if (dev >= 0 && dev < 64) configured[dev] = smem;
   }
-  MIE_CUDA(launch_chained(latent_decode_kernel<MT>, dim3(sm_count()), dim3(kLatentThreads), (size_t)smem, stream, map, p));
+  MIE_CUDA(launch_chained(latent_decode_kernel<MT, BOXES>, dim3(sm_count()), dim3(kLatentThreads), (size_t)smem, stream,
+                          map, p));
   MIE_LAUNCH_CHECK("latent_decode_kernel");
   return MIE_OK;
+}
+
+template <int MT>
+int launch_latent_boxes(const CUtensorMap& map, const LatentParams& p, cudaStream_t stream) {
+  if (p.key_boxes <= 4) return launch_latent<MT, 4>(map, p, stream);
+  if (p.key_boxes <= 9) return launch_latent<MT, 9>(map, p, stream);
+  return launch_latent<MT, kMaxKeyBoxes>(map, p, stream);
 }
 
 template <int VH>
@@ -475,7 +509,7 @@ extern "C" int mie_latent_decode_attention(const void* query, int64_t q_row_stri
                        IndexView(block_tables), IndexView(sequence_lengths), sc, batch, heads, block_size, num_blocks,
                        table_width, dim, value_dim, key_boxes, head_groups, slab ? 1 : 0, scale * 1.4426950408889634f,
                        window, sinks, status};
-  if (int rc = tiles == 1 ? launch_latent<1>(map, p, stream) : launch_latent<2>(map, p, stream)) return rc;
+  if (int rc = tiles == 1 ? launch_latent_boxes<1>(map, p, stream) : launch_latent_boxes<2>(map, p, stream)) return rc;
   mie_view4_t q{const_cast<void*>(query), {q_row_stride, q_head_stride, 0, 1}};
   mie_view4_t o{out, {o_row_stride, o_head_stride, 0, 1}};
   const DecodeParams merge{View4(q), View4(o), p.tables, p.lengths, IndexView(), sc, batch, heads, 1, heads, block_size,

@@ -86,19 +86,39 @@ __global__ void latent_write_kernel(LatentWriteParams p) {
   rotate_row<T>(row + p.q_rank + p.rank, slot + p.rank, p.rot_dim, p.rotated, p.turns, (float)pos, lane, 32);
 }
 
+// `lanes` lanes per token and group of heads; a lane turns one pair of every head of its group by the same angle.
+constexpr int kRotateHeads = 8;
+
 template <typename T>
 __global__ void rotate_heads_kernel(const T* src, long long s_token, long long s_head, T* dst, long long d_token,
                                     long long d_head, IndexView positions, const float2* turns, int tokens, int heads,
                                     int rot_dim, int rotated, int lanes) {
   chain_wait();
   chain_release();
-  const long long item = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
+  const long long t = ((long long)blockIdx.x * blockDim.x + threadIdx.x) / lanes;
   const int lane = threadIdx.x % lanes;
-  if (item >= (long long)tokens * heads) return;
-  const long long t = item / heads;
-  const int h = (int)(item % heads);
-  rotate_row<T>(src + t * s_token + h * s_head, dst + t * d_token + h * d_head, rot_dim, rotated, turns,
-                (float)positions.at(t), lane, lanes);
+  if (t >= tokens) return;
+  const float position = (float)positions.at(t);
+  const int h0 = blockIdx.y * kRotateHeads;
+  src += t * s_token + h0 * s_head;
+  dst += t * d_token + h0 * d_head;
+  heads = heads - h0 < kRotateHeads ? heads - h0 : kRotateHeads;
+  for (int i = lane; i < rotated / 2; i += lanes) {
+    float sine, cosine, u[kRotateHeads], v[kRotateHeads];  // all loads first: source and target may be the same rows
+#pragma unroll
+    for (int j = 0; j < kRotateHeads; ++j)
+      if (j < heads) u[j] = to_float<T>(src[j * s_head + 2 * i]), v[j] = to_float<T>(src[j * s_head + 2 * i + 1]);
+    turn_sincos(position, turns[i], &sine, &cosine);
+#pragma unroll
+    for (int j = 0; j < kRotateHeads; ++j)
+      if (j < heads) {
+        dst[j * d_head + 2 * i] = from_float<T>(u[j] * cosine - v[j] * sine);
+        dst[j * d_head + 2 * i + 1] = from_float<T>(v[j] * cosine + u[j] * sine);
+      }
+  }
+  if (dst != src)
+    for (int j = 0; j < heads; ++j)
+      for (int c = rotated + lane; c < rot_dim; c += lanes) dst[j * d_head + c] = src[j * s_head + c];
 }
 
 // spans: [requests] first row of a request's span in the gathered buffer, then [requests] its first token, then the
@@ -256,8 +276,8 @@ extern "C" int mie_rotate_heads(const void* src, int64_t src_token_stride, int64
   if (tokens == 0 || rot_dim == 0) return MIE_OK;
   int lanes = 1;
   while (lanes < 32 && lanes < (rot_dim + 1) / 2) lanes *= 2;
-  const long long threads = (long long)tokens * heads * lanes;
-  const dim3 grid((unsigned)((threads + 255) / 256)), block(256);
+  const long long threads = (long long)tokens * lanes;
+  const dim3 grid((unsigned)((threads + 127) / 128), (unsigned)((heads + kRotateHeads - 1) / kRotateHeads)), block(128);
   const float2* pairs = reinterpret_cast<const float2*>(turns);
   if (dtype == MIE_DTYPE_BF16)
     MIE_CUDA(launch_chained(rotate_heads_kernel<__nv_bfloat16>, grid, block, 0, (cudaStream_t)stream,

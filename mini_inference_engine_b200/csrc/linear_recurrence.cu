@@ -17,9 +17,7 @@
 namespace mie {
 namespace {
 
-__device__ __forceinline__ float sigmoid(float v) { return __fdividef(1.f, 1.f + expf(-v)); }
 __device__ __forceinline__ float silu(float v) { return __fdividef(v, 1.f + expf(-v)); }
-__device__ __forceinline__ float gru_candidate(float u) { return u >= 0.f ? u + 0.5f : sigmoid(u); }
 
 struct Slots {
   float* state;
@@ -194,27 +192,32 @@ __global__ void __launch_bounds__(kOuterWarps * 32) outer_rows_kernel(OuterParam
     for (int i = warp; i < p.dim; i += kOuterWarps) state[(long long)i * p.vdim] = tile[i * 32 + lane];
 }
 
-// The chunked form on tensor cores (bf16): one CTA per (segment, head, 64 value dims) walks its segment 64 tokens at
-// a time with the state in registers.  With q, k, v of 64 tokens and the state S before them,
+// The chunked form on tensor cores (bf16): one CTA per (segment, head, 64 * VD value dims) walks its segment 64 tokens
+// at a time with the state in registers.  With q, k, v of 64 tokens and the state S before them,
 //
-//   o_i  = decay^(i+1) S^T q_i + sum_(j <= i) decay^(i-j) (q_i . k_j) v_j
+//   o_i  = decay^(i+1) S^T q_i + sum_(j <= i) A_ij v_j,   A_ij = decay^(i-j) (q_i . k_j)
 //   S   <- decay^n S + sum_j k_j (decay^(n-1-j) v_j)^T
 //
-// q, k, v are the bf16 activations; S, the decayed products and the decayed v enter as a rounded part plus its
-// remainder (two MMAs), sums are fp32.  Four warps: warp w owns tokens 16w..16w+15 of the output and a quarter of the
-// key dims of the state.
+// q, k, v are the bf16 activations; S, A and the decayed v enter products as a rounded part plus its remainder (two
+// MMAs), sums are fp32.  The rows of the next tile are copied to a staging area while this one is computed; a thread
+// converts (silu) the 16-byte units it copied itself.  8 * VD warps: a warp computes 16 x (32 / VD) of A, 32 tokens x
+// 16 value dims of o, and 16 key dims x (KD * 32) value dims of the state.
 constexpr int kOuterTokens = 64;
-constexpr int kOuterCols = 64;
 
-template <int KD>  // 64-dim groups of a key row
+template <int KD, int VD>  // 64-dim groups of a key row, of a CTA's value row
 struct OuterTile {
+  static constexpr int kThreads = 256 * VD;
   static constexpr int kRow = 8192;  // 64 rows x 64 bf16, 128-byte rows, 16-byte units XOR-swizzled by row
   static constexpr int kOffQ = 0;
   static constexpr int kOffK = kOffQ + KD * kRow;
   static constexpr int kOffV = kOffK + KD * kRow;
-  static constexpr int kOffW = kOffV + kRow;           // decayed v: rounded part, remainder
-  static constexpr int kOffS = kOffW + 2 * kRow;       // state: rounded part, remainder
-  static constexpr int kOffPow = kOffS + 2 * KD * kRow;
+  static constexpr int kOffW = kOffV + VD * kRow;           // decayed v: rounded part, remainder
+  static constexpr int kOffS = kOffW + 2 * VD * kRow;       // state: rounded part, remainder; [key dim][value dim]
+  static constexpr int kOffA = kOffS + 2 * KD * VD * kRow;  // A: rounded part, remainder
+  static constexpr int kOffStage = kOffA + 2 * kRow;        // one 16-byte unit per thread and pass
+  static constexpr int kKeyPasses = kOuterTokens * KD * 8 / kThreads;
+  static constexpr int kValuePasses = kOuterTokens * VD * 8 / kThreads;
+  static constexpr int kOffPow = kOffStage + (2 * kKeyPasses + kValuePasses) * kThreads * 16;
   static constexpr int kSmem = kOffPow + 80 * 4;
 };
 
@@ -222,16 +225,32 @@ __device__ __forceinline__ uint32_t swizzled(int row, int unit) { return row * 1
 
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) { return Mma16816<__nv_bfloat16>::pack(lo, hi); }
 
-template <int KD, bool kEmit>
-__global__ void __launch_bounds__(128) outer_chunk_kernel(OuterParams p) {
-  using Tile = OuterTile<KD>;
+// silu of activations that are rounded to bf16 next.
+__device__ __forceinline__ float silu_rounded(float v) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(v * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
+  return v * r;
+}
+
+// 16 bytes global -> shared, or zeros.
+__device__ __forceinline__ void copy_async16(uint32_t dst, const void* src, bool live) {
+  asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
+}
+__device__ __forceinline__ void copy_async_commit() { asm volatile("cp.async.commit_group;" ::: "memory"); }
+__device__ __forceinline__ void copy_async_wait() { asm volatile("cp.async.wait_group 0;" ::: "memory"); }
+
+template <int KD, int VD, bool kEmit>
+__global__ void __launch_bounds__(256 * VD, KD + VD == 2 ? 2 : 1) outer_chunk_kernel(OuterParams p) {
+  using Tile = OuterTile<KD, VD>;
   using T = __nv_bfloat16;
   using Mma = Mma16816<T>;
+  constexpr int kThreads = Tile::kThreads, kRow = Tile::kRow;
   extern __shared__ __align__(1024) uint8_t chunk_smem[];
   float* powers = reinterpret_cast<float*>(chunk_smem + Tile::kOffPow);
   const uint32_t base = smem_u32(chunk_smem);
   const int tid = threadIdx.x, warp = tid >> 5, lane = tid & 31, g = lane >> 2, t4 = lane & 3;
-  const int h = blockIdx.y, col0 = blockIdx.z * kOuterCols;
+  const int h = blockIdx.y, col0 = blockIdx.z * VD * 64;
   chain_wait();
   chain_release();
   Segment seg;
@@ -242,8 +261,33 @@ __global__ void __launch_bounds__(128) outer_chunk_kernel(OuterParams p) {
   const float decay = p.decay[h];
   if (tid <= kOuterTokens) powers[tid] = powf(decay, (float)tid);
 
-  // State rows of this warp: m-tile mt covers key dims (warp * KD + mt) * 16 + {g, g + 8}.
-  float s[KD][8][4];
+  // Staging: passes of q, k, v units in turn, a thread's own unit of a pass at its own place.
+  auto stage = [&](long long tok0) {
+    const T* rows = reinterpret_cast<const T*>(p.rows);
+    uint32_t dst = base + Tile::kOffStage + tid * 16;
+#pragma unroll
+    for (int which = 0; which < 2; ++which)
+#pragma unroll
+      for (int pass = 0; pass < Tile::kKeyPasses; ++pass, dst += kThreads * 16) {
+        if (!kEmit && which == 0) continue;
+        const int i = pass * kThreads + tid, r = i / (KD * 8), unit = i % (KD * 8);
+        const bool live = tok0 + r < seg.end && unit * 8 < p.dim;
+        copy_async16(dst, rows + (live ? (tok0 + r) * p.ld + (which * p.heads + h) * p.dim + unit * 8 : 0), live);
+      }
+#pragma unroll
+    for (int pass = 0; pass < Tile::kValuePasses; ++pass, dst += kThreads * 16) {
+      const int i = pass * kThreads + tid, r = i / (VD * 8), unit = i % (VD * 8);
+      const bool live = tok0 + r < seg.end && col0 + unit * 8 < p.vdim;
+      copy_async16(dst, rows + (live ? (tok0 + r) * p.ld + 2 * p.heads * p.dim + h * p.vdim + col0 + unit * 8 : 0), live);
+    }
+    copy_async_commit();
+  };
+  stage(seg.begin);
+
+  // State tile of this warp: key dims s_row + {g, g + 8}, value dims s_col + nt * 8 + {2 t4, 2 t4 + 1}.
+  constexpr int kStateTiles = KD * 4;
+  float s[kStateTiles][4];
+  const int s_row = warp % (KD * 4) * 16, s_col = warp / (KD * 4) * (KD * 32);
   const long long head_state = (long long)h * p.dim * p.vdim;
   const long long carry_at = ((long long)blockIdx.x * p.heads + h) * p.dim * p.vdim;
   const float* init = nullptr;
@@ -255,12 +299,10 @@ __global__ void __launch_bounds__(128) outer_chunk_kernel(OuterParams p) {
   }
   auto each_pair = [&](auto&& visit) {  // two neighbouring columns of a state row
 #pragma unroll
-    for (int mt = 0; mt < KD; ++mt)
+    for (int nt = 0; nt < kStateTiles; ++nt)
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt)
-#pragma unroll
-        for (int half = 0; half < 2; ++half)
-          visit((warp * KD + mt) * 16 + g + half * 8, nt * 8 + 2 * t4, s[mt][nt][2 * half], s[mt][nt][2 * half + 1]);
+      for (int half = 0; half < 2; ++half)
+        visit(s_row + g + half * 8, s_col + nt * 8 + 2 * t4, s[nt][2 * half], s[nt][2 * half + 1]);
   };
   each_pair([&](int d, int c, float& a, float& b) {
     a = b = 0.f;
@@ -271,138 +313,146 @@ __global__ void __launch_bounds__(128) outer_chunk_kernel(OuterParams p) {
     }
   });
 
-  // ldmatrix lane geometry: plain B operand ([n][k] rows), transposed B operand ([k][n] rows), transposed A operand.
+  // ldmatrix lane geometry: plain B operand ([n][k] rows), transposed B operand ([k][n] rows), A operand, transposed A.
   const int b_row = (lane & 7) + ((lane >> 4) & 1) * 8, b_sel = (lane >> 3) & 1;
   const int v_row = (lane & 7) + ((lane >> 3) & 1) * 8, v_sel = (lane >> 4) & 1;
-  const int at_row = (lane & 7) + ((lane >> 4) & 1) * 8, at_sel = (lane >> 3) & 1;
-  const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_sel = (lane >> 4) & 1;
+  const int at_row = b_row, at_sel = b_sel;
+  const int a_row = v_row, a_sel = v_sel;
 
   for (long long tok0 = seg.begin; tok0 < seg.end; tok0 += kOuterTokens) {
     const int n = (int)(seg.end - tok0 < kOuterTokens ? seg.end - tok0 : kOuterTokens);
+    copy_async_wait();
     __syncthreads();  // the previous tile has been read (first pass: the powers are there)
-    const T* rows = reinterpret_cast<const T*>(p.rows) + tok0 * p.ld;
+    const uint8_t* staged = chunk_smem + Tile::kOffStage + tid * 16;
+    auto unpack = [&](float (&v)[8]) {
+      Vec<T, 8>::load(reinterpret_cast<const T*>(staged), v);
+#pragma unroll
+      for (int j = 0; j < 8; ++j) v[j] = silu_rounded(v[j]);
+      staged += kThreads * 16;
+    };
     // q and k through silu; rows past the segment and dims past the head are zero.
-    for (int i = tid; i < kOuterTokens * KD * 8; i += 128) {
-      const int r = i / (KD * 8), u = i % (KD * 8);
-      const bool in = r < n && u * 8 < p.dim;
-      uint32_t kq[2][4];
 #pragma unroll
-      for (int which = kEmit ? 0 : 1; which < 2; ++which) {
+    for (int which = 0; which < 2; ++which) {
+      if (!kEmit && which == 0) {
+        staged += Tile::kKeyPasses * kThreads * 16;
+        continue;
+      }
+#pragma unroll
+      for (int pass = 0; pass < Tile::kKeyPasses; ++pass) {
+        const int i = pass * kThreads + tid, r = i / (KD * 8), unit = i % (KD * 8);
         float v[8];
-        if (in) {
-          Vec<T, 8>::load(rows + (long long)r * p.ld + (which * p.heads + h) * p.dim + u * 8, v);
-        } else {
-#pragma unroll
-          for (int j = 0; j < 8; ++j) v[j] = 0.f;
-        }
-#pragma unroll
-        for (int j = 0; j < 4; ++j) kq[which][j] = pack_bf16(silu(v[2 * j]), silu(v[2 * j + 1]));
-        *reinterpret_cast<uint4*>(chunk_smem + (which == 0 ? Tile::kOffQ : Tile::kOffK) + (u >> 3) * Tile::kRow +
-                                  swizzled(r, u & 7)) =
-            make_uint4(kq[which][0], kq[which][1], kq[which][2], kq[which][3]);
+        unpack(v);
+        *reinterpret_cast<uint4*>(chunk_smem + (which == 0 ? Tile::kOffQ : Tile::kOffK) + (unit >> 3) * kRow +
+                                  swizzled(r, unit & 7)) =
+            make_uint4(pack_bf16(v[0], v[1]), pack_bf16(v[2], v[3]), pack_bf16(v[4], v[5]), pack_bf16(v[6], v[7]));
       }
     }
-    for (int i = tid; i < kOuterTokens * 8; i += 128) {
-      const int r = i / 8, u = i % 8;
-      float v[8];
-      if (r < n && col0 + u * 8 < p.vdim) {
-        Vec<T, 8>::load(rows + (long long)r * p.ld + 2 * p.heads * p.dim + h * p.vdim + col0 + u * 8, v);
-      } else {
 #pragma unroll
-        for (int j = 0; j < 8; ++j) v[j] = 0.f;
-      }
+    for (int pass = 0; pass < Tile::kValuePasses; ++pass) {
+      const int i = pass * kThreads + tid, r = i / (VD * 8), unit = i % (VD * 8);
+      float v[8];
+      unpack(v);
       const float weight = r < n ? powers[n - 1 - r] : 0.f;
       uint32_t whole[4], high[4], low[4];
 #pragma unroll
       for (int j = 0; j < 4; ++j) {
-        const float a = round_bf16(silu(v[2 * j])), b = round_bf16(silu(v[2 * j + 1]));
-        const float wa = a * weight, wb = b * weight;
-        whole[j] = pack_bf16(a, b);
+        whole[j] = pack_bf16(v[2 * j], v[2 * j + 1]);
+        const float2 b = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&whole[j]));
+        const float wa = b.x * weight, wb = b.y * weight;
         high[j] = pack_bf16(wa, wb);
-        low[j] = pack_bf16(wa - round_bf16(wa), wb - round_bf16(wb));
+        const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&high[j]));
+        low[j] = pack_bf16(wa - k.x, wb - k.y);
       }
-      const uint32_t off = swizzled(r, u);
-      *reinterpret_cast<uint4*>(chunk_smem + Tile::kOffV + off) = make_uint4(whole[0], whole[1], whole[2], whole[3]);
+      const uint32_t off = (unit >> 3) * kRow + swizzled(r, unit & 7);
+      if (kEmit) *reinterpret_cast<uint4*>(chunk_smem + Tile::kOffV + off) = make_uint4(whole[0], whole[1], whole[2], whole[3]);
       *reinterpret_cast<uint4*>(chunk_smem + Tile::kOffW + off) = make_uint4(high[0], high[1], high[2], high[3]);
-      *reinterpret_cast<uint4*>(chunk_smem + Tile::kOffW + Tile::kRow + off) = make_uint4(low[0], low[1], low[2], low[3]);
+      *reinterpret_cast<uint4*>(chunk_smem + Tile::kOffW + VD * kRow + off) = make_uint4(low[0], low[1], low[2], low[3]);
     }
+    if (tok0 + kOuterTokens < seg.end) stage(tok0 + kOuterTokens);
     if (kEmit) {
       each_pair([&](int d, int c, float& a, float& b) {
-        const uint32_t off = (d >> 6) * Tile::kRow + swizzled(d & 63, c >> 3) + (c & 7) * 2;
-        *reinterpret_cast<uint32_t*>(chunk_smem + Tile::kOffS + off) = pack_bf16(a, b);
-        *reinterpret_cast<uint32_t*>(chunk_smem + Tile::kOffS + KD * Tile::kRow + off) =
-            pack_bf16(a - round_bf16(a), b - round_bf16(b));
+        const uint32_t off = ((d >> 6) * VD + (c >> 6)) * kRow + swizzled(d & 63, (c & 63) >> 3) + (c & 7) * 2;
+        const uint32_t high = pack_bf16(a, b);
+        const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&high));
+        *reinterpret_cast<uint32_t*>(chunk_smem + Tile::kOffS + off) = high;
+        *reinterpret_cast<uint32_t*>(chunk_smem + Tile::kOffS + KD * VD * kRow + off) = pack_bf16(a - k.x, b - k.y);
       });
     }
     __syncthreads();
 
-    if (kEmit && warp * 16 < n) {
-      float o[8][4], a[8][4];
+    float o[2][2][4];  // tokens o_tok + mt * 16 + {g, g + 8}, value dims o_col + nt * 8 + ...
+    const int o_tok = (warp & 1) * 32, o_col = (warp >> 1) * 16;
+    const uint32_t o_group = (o_col >> 6) * kRow;
+    const int o_unit = (o_col & 63) >> 3;
+    if (kEmit) {
+      // A: tokens 16 (warp & 3) ..., keys from block j_blk on; blocks above the diagonal are never read.
+      constexpr int kBlocks = 2 / VD;
+      const int i_blk = warp & 3, j_blk = (warp >> 2) * kBlocks;
+      if (j_blk <= i_blk) {
+        float a[2 * kBlocks][4];
 #pragma unroll
-      for (int i = 0; i < 8; ++i)
+        for (int i = 0; i < 2 * kBlocks; ++i) a[i][0] = a[i][1] = a[i][2] = a[i][3] = 0.f;
 #pragma unroll
-        for (int j = 0; j < 4; ++j) o[i][j] = a[i][j] = 0.f;
+        for (int ks = 0; ks < KD * 4; ++ks) {
+          const uint32_t group = (ks >> 2) * kRow;
+          uint32_t q[4], r[4];
+          ldmatrix_x4(q[0], q[1], q[2], q[3],
+                      base + Tile::kOffQ + group + swizzled(i_blk * 16 + a_row, (ks & 3) * 2 + a_sel));
+#pragma unroll
+          for (int np = 0; np < kBlocks; ++np) {
+            if (np > 0 && j_blk + np > i_blk) break;
+            ldmatrix_x4(r[0], r[1], r[2], r[3],
+                        base + Tile::kOffK + group + swizzled((j_blk + np) * 16 + b_row, (ks & 3) * 2 + b_sel));
+            Mma::run(a[2 * np], q[0], q[1], q[2], q[3], r[0], r[1]);
+            Mma::run(a[2 * np + 1], q[0], q[1], q[2], q[3], r[2], r[3]);
+          }
+        }
+        const int i0 = i_blk * 16 + g;
+#pragma unroll
+        for (int nt = 0; nt < 2 * kBlocks; ++nt) {
+          const int j = j_blk * 16 + nt * 8 + 2 * t4;
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int i = i0 + e * 8;
+            const float x = i >= j ? a[nt][2 * e] * powers[i - j] : 0.f;
+            const float y = i >= j + 1 ? a[nt][2 * e + 1] * powers[i - j - 1] : 0.f;
+            const uint32_t off = Tile::kOffA + swizzled(i, j >> 3) + (j & 7) * 2, high = pack_bf16(x, y);
+            const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&high));
+            *reinterpret_cast<uint32_t*>(chunk_smem + off) = high;
+            *reinterpret_cast<uint32_t*>(chunk_smem + off + kRow) = pack_bf16(x - k.x, y - k.y);
+          }
+        }
+      }
+      // S^T q.
+#pragma unroll
+      for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) o[mt][nt][0] = o[mt][nt][1] = o[mt][nt][2] = o[mt][nt][3] = 0.f;
 #pragma unroll
       for (int ks = 0; ks < KD * 4; ++ks) {
-        if (ks * 16 >= p.dim) break;
-        const uint32_t group = (ks >> 2) * Tile::kRow;
-        uint32_t q0, q1, q2, q3;
-        ldmatrix_x4(q0, q1, q2, q3, base + Tile::kOffQ + group + swizzled(warp * 16 + a_row, (ks & 3) * 2 + a_sel));
+        uint32_t q[2][4];
 #pragma unroll
-        for (int np = 0; np < 4; ++np) {
-          uint32_t r0, r1, r2, r3;
-          if (np <= warp) {  // q . k, tokens up to this warp's
-            ldmatrix_x4(r0, r1, r2, r3, base + Tile::kOffK + group + swizzled(np * 16 + b_row, (ks & 3) * 2 + b_sel));
-            Mma::run(a[2 * np], q0, q1, q2, q3, r0, r1);
-            Mma::run(a[2 * np + 1], q0, q1, q2, q3, r2, r3);
-          }
+        for (int mt = 0; mt < 2; ++mt)
+          ldmatrix_x4(q[mt][0], q[mt][1], q[mt][2], q[mt][3],
+                      base + Tile::kOffQ + (ks >> 2) * kRow + swizzled(o_tok + mt * 16 + a_row, (ks & 3) * 2 + a_sel));
 #pragma unroll
-          for (int part = 0; part < 2; ++part) {  // S^T q
-            ldmatrix_x4_trans(r0, r1, r2, r3, base + Tile::kOffS + part * KD * Tile::kRow + group +
-                                                  swizzled((ks & 3) * 16 + v_row, np * 2 + v_sel));
-            Mma::run(o[2 * np], q0, q1, q2, q3, r0, r1);
-            Mma::run(o[2 * np + 1], q0, q1, q2, q3, r2, r3);
+        for (int part = 0; part < 2; ++part) {
+          uint32_t r[4];
+          ldmatrix_x4_trans(r[0], r[1], r[2], r[3],
+                            base + Tile::kOffS + (part * KD + (ks >> 2)) * VD * kRow + o_group +
+                                swizzled((ks & 3) * 16 + v_row, o_unit + v_sel));
+#pragma unroll
+          for (int mt = 0; mt < 2; ++mt) {
+            Mma::run(o[mt][0], q[mt][0], q[mt][1], q[mt][2], q[mt][3], r[0], r[1]);
+            Mma::run(o[mt][1], q[mt][0], q[mt][1], q[mt][2], q[mt][3], r[2], r[3]);
           }
         }
       }
-      const int i0 = warp * 16 + g, i1 = i0 + 8;
-      const float d0 = powers[i0 + 1], d1 = powers[i1 + 1];
 #pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        o[nt][0] *= d0, o[nt][1] *= d0, o[nt][2] *= d1, o[nt][3] *= d1;
-        const int j = nt * 8 + 2 * t4;
-        a[nt][0] = i0 >= j ? a[nt][0] * powers[i0 - j] : 0.f;
-        a[nt][1] = i0 >= j + 1 ? a[nt][1] * powers[i0 - j - 1] : 0.f;
-        a[nt][2] = i1 >= j ? a[nt][2] * powers[i1 - j] : 0.f;
-        a[nt][3] = i1 >= j + 1 ? a[nt][3] * powers[i1 - j - 1] : 0.f;
-      }
+      for (int mt = 0; mt < 2; ++mt) {
+        const float d0 = powers[o_tok + mt * 16 + g + 1], d1 = powers[o_tok + mt * 16 + g + 9];
 #pragma unroll
-      for (int kt = 0; kt < 4; ++kt) {
-        if (kt > warp) break;
-        uint32_t hi[4], lo[4];
-#pragma unroll
-        for (int e = 0; e < 4; ++e) {
-          const float x = a[2 * kt + (e >> 1)][(e & 1) * 2], y = a[2 * kt + (e >> 1)][(e & 1) * 2 + 1];
-          hi[e] = pack_bf16(x, y);
-          lo[e] = pack_bf16(x - round_bf16(x), y - round_bf16(y));
-        }
-#pragma unroll
-        for (int np = 0; np < 4; ++np) {
-          uint32_t r0, r1, r2, r3;
-          ldmatrix_x4_trans(r0, r1, r2, r3, base + Tile::kOffV + swizzled(kt * 16 + v_row, np * 2 + v_sel));
-          Mma::run(o[2 * np], hi[0], hi[1], hi[2], hi[3], r0, r1);
-          Mma::run(o[2 * np + 1], hi[0], hi[1], hi[2], hi[3], r2, r3);
-          Mma::run(o[2 * np], lo[0], lo[1], lo[2], lo[3], r0, r1);
-          Mma::run(o[2 * np + 1], lo[0], lo[1], lo[2], lo[3], r2, r3);
-        }
-      }
-      T* out = reinterpret_cast<T*>(p.out) + tok0 * p.ldo + h * p.vdim + col0;
-#pragma unroll
-      for (int nt = 0; nt < 8; ++nt) {
-        const int c = nt * 8 + 2 * t4;
-        if (col0 + c >= p.vdim) break;
-        if (i0 < n) *reinterpret_cast<uint32_t*>(out + (long long)i0 * p.ldo + c) = pack_bf16(o[nt][0], o[nt][1]);
-        if (i1 < n) *reinterpret_cast<uint32_t*>(out + (long long)i1 * p.ldo + c) = pack_bf16(o[nt][2], o[nt][3]);
+        for (int nt = 0; nt < 2; ++nt) o[mt][nt][0] *= d0, o[mt][nt][1] *= d0, o[mt][nt][2] *= d1, o[mt][nt][3] *= d1;
       }
     }
 
@@ -415,24 +465,56 @@ __global__ void __launch_bounds__(128) outer_chunk_kernel(OuterParams p) {
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
       if (kt * 16 >= n) break;
-      uint32_t ka[KD][4];
+      uint32_t ka[4];
+      const int unit = (s_row >> 3) + at_sel;  // 16-byte unit of the key row
+      ldmatrix_x4_trans(ka[0], ka[1], ka[2], ka[3],
+                        base + Tile::kOffK + (unit >> 3) * kRow + swizzled(kt * 16 + at_row, unit & 7));
 #pragma unroll
-      for (int mt = 0; mt < KD; ++mt) {
-        const int unit = (warp * KD + mt) * 2 + at_sel;  // 16-byte unit of the key row
-        ldmatrix_x4_trans(ka[mt][0], ka[mt][1], ka[mt][2], ka[mt][3],
-                          base + Tile::kOffK + (unit >> 3) * Tile::kRow + swizzled(kt * 16 + at_row, unit & 7));
-      }
-#pragma unroll
-      for (int np = 0; np < 4; ++np)
+      for (int np = 0; np < kStateTiles / 2; ++np)
 #pragma unroll
         for (int part = 0; part < 2; ++part) {
-          uint32_t r0, r1, r2, r3;
-          ldmatrix_x4_trans(r0, r1, r2, r3,
-                            base + Tile::kOffW + part * Tile::kRow + swizzled(kt * 16 + v_row, np * 2 + v_sel));
+          const int c = s_col + np * 16;
+          uint32_t r[4];
+          ldmatrix_x4_trans(r[0], r[1], r[2], r[3],
+                            base + Tile::kOffW + (part * VD + (c >> 6)) * kRow +
+                                swizzled(kt * 16 + v_row, ((c & 63) >> 3) + v_sel));
+          Mma::run(s[2 * np], ka[0], ka[1], ka[2], ka[3], r[0], r[1]);
+          Mma::run(s[2 * np + 1], ka[0], ka[1], ka[2], ka[3], r[2], r[3]);
+        }
+    }
+
+    if (kEmit) {
+      __syncthreads();  // A is complete
 #pragma unroll
-          for (int mt = 0; mt < KD; ++mt) {
-            Mma::run(s[mt][2 * np], ka[mt][0], ka[mt][1], ka[mt][2], ka[mt][3], r0, r1);
-            Mma::run(s[mt][2 * np + 1], ka[mt][0], ka[mt][1], ka[mt][2], ka[mt][3], r2, r3);
+      for (int kt = 0; kt < 4; ++kt) {
+        if (kt * 16 > o_tok + 16) break;
+        uint32_t r[4];
+        ldmatrix_x4_trans(r[0], r[1], r[2], r[3], base + Tile::kOffV + o_group + swizzled(kt * 16 + v_row, o_unit + v_sel));
+#pragma unroll
+        for (int mt = 0; mt < 2; ++mt) {
+          if (kt * 16 > o_tok + mt * 16) continue;  // above the diagonal
+#pragma unroll
+          for (int part = 0; part < 2; ++part) {
+            uint32_t a[4];
+            ldmatrix_x4(a[0], a[1], a[2], a[3],
+                        base + Tile::kOffA + part * kRow + swizzled(o_tok + mt * 16 + a_row, kt * 2 + a_sel));
+            Mma::run(o[mt][0], a[0], a[1], a[2], a[3], r[0], r[1]);
+            Mma::run(o[mt][1], a[0], a[1], a[2], a[3], r[2], r[3]);
+          }
+        }
+      }
+      T* out = reinterpret_cast<T*>(p.out) + tok0 * p.ldo + h * p.vdim + col0;
+#pragma unroll
+      for (int mt = 0; mt < 2; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < 2; ++nt) {
+          const int c = o_col + nt * 8 + 2 * t4;
+          if (col0 + c >= p.vdim) continue;
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int i = o_tok + mt * 16 + g + e * 8;
+            if (i < n)
+              *reinterpret_cast<uint32_t*>(out + (long long)i * p.ldo + c) = pack_bf16(o[mt][nt][2 * e], o[mt][nt][2 * e + 1]);
           }
         }
     }
@@ -445,6 +527,8 @@ __global__ void __launch_bounds__(128) outer_chunk_kernel(OuterParams p) {
       *reinterpret_cast<float2*>(dst + (long long)d * p.vdim + col0 + c) = make_float2(a, b);
   });
 }
+
+constexpr int kCarryBatch = 8;  // segments whose loads are in flight together
 
 // carry[segment] <- state before the segment, from what the segments before it added.
 __global__ void outer_carry_kernel(OuterParams p) {
@@ -465,11 +549,18 @@ __global__ void outer_carry_kernel(OuterParams p) {
   if (slot == nullptr) return;
   float state = p.positions.at(begin) == 0 ? 0.f : slot[(long long)h * size + e];
   const float decay = powf(p.decay[h], (float)p.seg.length);
-  for (int i = 0; i < pieces; ++i) {
-    float* at = p.carry + ((long long)(first + i) * p.heads + h) * size + e;
-    const float added = i + 1 < pieces ? *at : 0.f;
-    *at = state;
-    state = decay * state + added;
+  const long long stride = (long long)p.heads * size;
+  float* at = p.carry + (long long)first * stride + (long long)h * size + e;
+  for (int i0 = 0; i0 < pieces; i0 += kCarryBatch, at += kCarryBatch * stride) {
+    float added[kCarryBatch];
+#pragma unroll
+    for (int i = 0; i < kCarryBatch; ++i) added[i] = i0 + i + 1 < pieces ? at[i * stride] : 0.f;
+#pragma unroll
+    for (int i = 0; i < kCarryBatch; ++i) {
+      if (i0 + i >= pieces) break;
+      at[i * stride] = state;
+      state = decay * state + added[i];
+    }
   }
 }
 
@@ -490,6 +581,16 @@ struct AverageParams {
   float* carry;  // [segments][2][width], null: every request is one segment
 };
 
+// keep = 1 - z, add = z * candidate.  The two sigmoids share one reciprocal; their exponents are bounded so that the
+// product of the denominators stays finite (a sigmoid below 1e-17 is 1e-17).
+__device__ __forceinline__ void average_gates(float a, float u, float* keep, float* add) {
+  const float da = 1.f + expf(fminf(-a, 40.f)), du = 1.f + expf(fminf(-u, 40.f));
+  const float inv = __fdividef(1.f, da * du);
+  const float gate = inv * du;
+  *keep = 1.f - gate;
+  *add = gate * (u >= 0.f ? u + 0.5f : inv * da);
+}
+
 template <typename T, int VEC>
 struct AverageStep {
   float zb[VEC], ub[VEC];
@@ -497,27 +598,32 @@ struct AverageStep {
     Vec<T, VEC>::load(reinterpret_cast<const T*>(p.z_bias) + c, zb);
     Vec<T, VEC>::load(reinterpret_cast<const T*>(p.u_bias) + c, ub);
   }
-  // keep = 1 - z, add = z * candidate
-  __device__ __forceinline__ void gates(const T* row, int width, float (&keep)[VEC], float (&add)[VEC]) const {
-    float z[VEC], u[VEC];
-    Vec<T, VEC>::load(row, z);
-    Vec<T, VEC>::load(row + width, u);
+  __device__ __forceinline__ void gates(const float (&z)[VEC], const float (&u)[VEC], float (&keep)[VEC],
+                                        float (&add)[VEC]) const {
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-      const float gate = sigmoid(z[j] + zb[j]);
-      keep[j] = 1.f - gate;
-      add[j] = gate * gru_candidate(u[j] + ub[j]);
-    }
+    for (int j = 0; j < VEC; ++j) average_gates(z[j] + zb[j], u[j] + ub[j], &keep[j], &add[j]);
+  }
+};
+constexpr int kAverageBatch = 4;  // tokens whose loads are in flight together
+
+// VEC activations as they lie in memory, widened when they are used.
+template <typename T, int VEC>
+struct alignas(sizeof(T) * VEC) RawVec {
+  T v[VEC];
+  __device__ __forceinline__ static RawVec at(const T* p) { return *reinterpret_cast<const RawVec*>(p); }
+  __device__ __forceinline__ void widen(float (&out)[VEC]) const {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) out[j] = to_float<T>(v[j]);
   }
 };
 
+// state * silu(g)
 template <typename T, int VEC>
-__device__ __forceinline__ void average_emit(const T* row, int width, T* out, const float (&state)[VEC]) {
-  float g[VEC];
-  Vec<T, VEC>::load(row + 2 * width, g);
+__device__ __forceinline__ void average_emit(const float (&g)[VEC], T* out, const float (&state)[VEC]) {
+  float v[VEC];
 #pragma unroll
-  for (int j = 0; j < VEC; ++j) g[j] = state[j] * silu(g[j]);
-  Vec<T, VEC>::store(out, g);
+  for (int j = 0; j < VEC; ++j) v[j] = state[j] * silu(g[j]);
+  Vec<T, VEC>::store(out, v);
 }
 
 template <typename T, int VEC>
@@ -530,23 +636,26 @@ __global__ void average_decode_kernel(AverageParams p) {
   if (slot == nullptr) return;
   const T* src = reinterpret_cast<const T*>(p.rows) + (long long)row * p.ld + c;
   const AverageStep<T, VEC> step(p, c);
-  float state[VEC], keep[VEC], add[VEC];
+  float state[VEC], keep[VEC], add[VEC], z[VEC], u[VEC], g[VEC];
+  Vec<T, VEC>::load(src, z);
+  Vec<T, VEC>::load(src + p.width, u);
+  Vec<T, VEC>::load(src + 2 * p.width, g);
   if (p.positions.at(row) == 0) {
 #pragma unroll
     for (int j = 0; j < VEC; ++j) state[j] = 0.f;
   } else {
     Vec<float, VEC>::load(slot + c, state);
   }
-  step.gates(src, p.width, keep, add);
+  step.gates(z, u, keep, add);
 #pragma unroll
   for (int j = 0; j < VEC; ++j) state[j] = keep[j] * state[j] + add[j];
   Vec<float, VEC>::store(slot + c, state);
-  average_emit<T, VEC>(src, p.width, reinterpret_cast<T*>(p.out) + (long long)row * p.ldo + c, state);
+  average_emit<T, VEC>(g, reinterpret_cast<T*>(p.out) + (long long)row * p.ldo + c, state);
 }
 
 // What a segment does to a state before it: S -> product S + sum.
 template <typename T, int VEC>
-__global__ void average_summary_kernel(AverageParams p) {
+__global__ void __launch_bounds__(128, 6) average_summary_kernel(AverageParams p) {
   chain_wait();
   chain_release();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
@@ -557,14 +666,27 @@ __global__ void average_summary_kernel(AverageParams p) {
 #pragma unroll
   for (int j = 0; j < VEC; ++j) product[j] = 1.f, sum[j] = 0.f;
   const T* src = reinterpret_cast<const T*>(p.rows) + seg.begin * p.ld + c;
-#pragma unroll 8
-  for (long long t = seg.begin; t < seg.end; ++t, src += p.ld) {
-    float keep[VEC], add[VEC];
-    step.gates(src, p.width, keep, add);
+  const int count = (int)(seg.end - seg.begin);
+  for (int t0 = 0; t0 < count; t0 += kAverageBatch, src += kAverageBatch * p.ld) {
+    RawVec<T, VEC> z[kAverageBatch], u[kAverageBatch];
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-      product[j] *= keep[j];
-      sum[j] = keep[j] * sum[j] + add[j];
+    for (int i = 0; i < kAverageBatch; ++i)
+      if (t0 + i < count) {
+        z[i] = RawVec<T, VEC>::at(src + i * p.ld);
+        u[i] = RawVec<T, VEC>::at(src + i * p.ld + p.width);
+      }
+#pragma unroll
+    for (int i = 0; i < kAverageBatch; ++i) {
+      if (t0 + i >= count) break;
+      float keep[VEC], add[VEC], a[VEC], b[VEC];
+      z[i].widen(a);
+      u[i].widen(b);
+      step.gates(a, b, keep, add);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        product[j] *= keep[j];
+        sum[j] = keep[j] * sum[j] + add[j];
+      }
     }
   }
   float* dst = p.carry + (long long)blockIdx.x * 2 * p.width + c;
@@ -590,16 +712,25 @@ __global__ void average_carry_kernel(AverageParams p) {
   if (slot == nullptr) return;
   float state = p.positions.at(begin) == 0 ? 0.f : slot[c];
   float* at = p.carry + (long long)first * 2 * p.width + c;
-#pragma unroll 8
-  for (int i = 0; i < pieces; ++i, at += 2 * p.width) {
-    const float product = i + 1 < pieces ? at[0] : 0.f, sum = i + 1 < pieces ? at[p.width] : 0.f;
-    at[0] = state;
-    state = product * state + sum;
+  for (int i0 = 0; i0 < pieces; i0 += kCarryBatch, at += (long long)kCarryBatch * 2 * p.width) {
+    float product[kCarryBatch], sum[kCarryBatch];
+#pragma unroll
+    for (int i = 0; i < kCarryBatch; ++i) {
+      const bool more = i0 + i + 1 < pieces;
+      product[i] = more ? at[(long long)i * 2 * p.width] : 0.f;
+      sum[i] = more ? at[(long long)i * 2 * p.width + p.width] : 0.f;
+    }
+#pragma unroll
+    for (int i = 0; i < kCarryBatch; ++i) {
+      if (i0 + i >= pieces) break;
+      at[(long long)i * 2 * p.width] = state;
+      state = product[i] * state + sum[i];
+    }
   }
 }
 
 template <typename T, int VEC>
-__global__ void average_segment_kernel(AverageParams p) {
+__global__ void __launch_bounds__(128, 6) average_segment_kernel(AverageParams p) {
   chain_wait();
   chain_release();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
@@ -619,13 +750,28 @@ __global__ void average_segment_kernel(AverageParams p) {
   }
   const T* src = reinterpret_cast<const T*>(p.rows) + seg.begin * p.ld + c;
   T* out = reinterpret_cast<T*>(p.out) + seg.begin * p.ldo + c;
-#pragma unroll 4
-  for (long long t = seg.begin; t < seg.end; ++t, src += p.ld, out += p.ldo) {
-    float keep[VEC], add[VEC];
-    step.gates(src, p.width, keep, add);
+  const int count = (int)(seg.end - seg.begin);
+  for (int t0 = 0; t0 < count; t0 += kAverageBatch, src += kAverageBatch * p.ld, out += kAverageBatch * p.ldo) {
+    RawVec<T, VEC> z[kAverageBatch], u[kAverageBatch], g[kAverageBatch];
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) state[j] = keep[j] * state[j] + add[j];
-    average_emit<T, VEC>(src, p.width, out, state);
+    for (int i = 0; i < kAverageBatch; ++i)
+      if (t0 + i < count) {
+        z[i] = RawVec<T, VEC>::at(src + i * p.ld);
+        u[i] = RawVec<T, VEC>::at(src + i * p.ld + p.width);
+        g[i] = RawVec<T, VEC>::at(src + i * p.ld + 2 * p.width);
+      }
+#pragma unroll
+    for (int i = 0; i < kAverageBatch; ++i) {
+      if (t0 + i >= count) break;
+      float keep[VEC], add[VEC], a[VEC], b[VEC];
+      z[i].widen(a);
+      u[i].widen(b);
+      step.gates(a, b, keep, add);
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) state[j] = keep[j] * state[j] + add[j];
+      g[i].widen(a);
+      average_emit<T, VEC>(a, out + i * p.ldo, state);
+    }
   }
   if (seg.last) Vec<float, VEC>::store(slot + c, state);
 }
@@ -659,20 +805,21 @@ int launch_outer_rows(const OuterParams& p, cudaStream_t stream) {
   return MIE_OK;
 }
 
-template <int KD>
+template <int KD, int VD>
 int launch_outer_chunks(const OuterParams& p, int segments, cudaStream_t stream) {
-  constexpr int smem = OuterTile<KD>::kSmem;
-  const dim3 grid((unsigned)segments, (unsigned)p.heads, (unsigned)((p.vdim + kOuterCols - 1) / kOuterCols));
+  constexpr int smem = OuterTile<KD, VD>::kSmem;
+  const dim3 grid((unsigned)segments, (unsigned)p.heads, (unsigned)((p.vdim + VD * 64 - 1) / (VD * 64)));
+  const dim3 block(OuterTile<KD, VD>::kThreads);
   if (p.carry != nullptr) {
-    if (int rc = allow_smem(outer_chunk_kernel<KD, false>, smem)) return rc;
-    MIE_CUDA(launch_chained(outer_chunk_kernel<KD, false>, grid, dim3(128), (size_t)smem, stream, p));
+    if (int rc = allow_smem(outer_chunk_kernel<KD, VD, false>, smem)) return rc;
+    MIE_CUDA(launch_chained(outer_chunk_kernel<KD, VD, false>, grid, block, (size_t)smem, stream, p));
     MIE_LAUNCH_CHECK("outer_chunk_kernel");
     const dim3 flat((unsigned)(p.seg.requests * p.heads), (unsigned)((p.dim * p.vdim + 255) / 256));
     MIE_CUDA(launch_chained(outer_carry_kernel, flat, dim3(256), 0, stream, p));
     MIE_LAUNCH_CHECK("outer_carry_kernel");
   }
-  if (int rc = allow_smem(outer_chunk_kernel<KD, true>, smem)) return rc;
-  MIE_CUDA(launch_chained(outer_chunk_kernel<KD, true>, grid, dim3(128), (size_t)smem, stream, p));
+  if (int rc = allow_smem(outer_chunk_kernel<KD, VD, true>, smem)) return rc;
+  MIE_CUDA(launch_chained(outer_chunk_kernel<KD, VD, true>, grid, block, (size_t)smem, stream, p));
   MIE_LAUNCH_CHECK("outer_chunk_kernel");
   return MIE_OK;
 }
@@ -770,7 +917,9 @@ extern "C" int mie_outer_recurrence(const void* rows, int64_t ld, const float* d
   } else {
     p.seg.length = 0x40000000;
   }
-  return dim <= 64 ? launch_outer_chunks<1>(p, segments, stream) : launch_outer_chunks<2>(p, segments, stream);
+  if (value_dim <= 64)
+    return dim <= 64 ? launch_outer_chunks<1, 1>(p, segments, stream) : launch_outer_chunks<2, 1>(p, segments, stream);
+  return dim <= 64 ? launch_outer_chunks<1, 2>(p, segments, stream) : launch_outer_chunks<2, 2>(p, segments, stream);
 }
 
 extern "C" int mie_gated_average(const void* rows, int64_t ld, const void* z_bias, const void* u_bias, void* out,

@@ -25,8 +25,12 @@ struct ResidualParams {
   float eps;
 };
 
+// A thread's first kKept groups of VEC entries, one block width apart, stay in registers with their operands, which
+// are all fetched before the first reduction; wider rows are read again.
+constexpr int kKept = 2;
+
 template <typename T, int VEC>
-__global__ void __launch_bounds__(1024) residual_norm_kernel(ResidualParams p) {
+__global__ void __launch_bounds__(512) residual_norm_kernel(ResidualParams p) {
   __shared__ float red[2][32];
   chain_wait();
   chain_release();
@@ -34,51 +38,59 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(ResidualParams p) {
   float* x = p.x + (long long)blockIdx.x * p.ldx;
   const T* y = reinterpret_cast<const T*>(p.y) + (long long)blockIdx.x * p.ldy;
   const T* yw = reinterpret_cast<const T*>(p.y_weight);
-  // A thread's first group stays in registers; rows wider than one sweep are read again.
-  float kept[VEC];
+  const T* nw = p.out == nullptr ? nullptr : reinterpret_cast<const T*>(p.next_weight);
+  float sums[kKept][VEC], ys[kKept][VEC], yws[kKept][VEC];
   float ss = 0.f;
-  for (int c = tid * VEC; c < p.cols; c += step) {
+#pragma unroll
+  for (int k = 0; k < kKept; ++k) {
+    const int c = (k * blockDim.x + tid) * VEC;
+    if (c < p.cols) {
+      Vec<T, VEC>::load(y + c, ys[k]);
+      Vec<float, VEC>::load(x + c, sums[k]);
+      Vec<T, VEC>::load(yw + c, yws[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kKept; ++k)
+    if ((k * (int)blockDim.x + tid) * VEC < p.cols)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ss += ys[k][j] * ys[k][j];
+  for (int c = (kKept * blockDim.x + tid) * VEC; c < p.cols; c += step) {
     float v[VEC];
     Vec<T, VEC>::load(y + c, v);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-      ss += v[j] * v[j];
-      if (c < step) kept[j] = v[j];
+    for (int j = 0; j < VEC; ++j) ss += v[j] * v[j];
+  }
+  const float inv_y = p.alpha / sqrtf(block_sum(ss, red[0]) / (float)p.cols + p.eps);
+  ss = 0.f;
+#pragma unroll
+  for (int k = 0; k < kKept; ++k) {
+    const int c = (k * blockDim.x + tid) * VEC;
+    if (c < p.cols) {
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) {
+        sums[k][j] += ys[k][j] * inv_y * yws[k][j];
+        ss += sums[k][j] * sums[k][j];
+      }
+      Vec<float, VEC>::store(x + c, sums[k]);
     }
   }
-  const float inv_y = 1.f / sqrtf(block_sum(ss, red[0]) / (float)p.cols + p.eps);
-  ss = 0.f;
-  for (int c = tid * VEC; c < p.cols; c += step) {
+  for (int c = (kKept * blockDim.x + tid) * VEC; c < p.cols; c += step) {
     float v[VEC], w[VEC], r[VEC];
-    if (c < step) {
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) v[j] = kept[j];
-    } else {
-      Vec<T, VEC>::load(y + c, v);
-    }
+    Vec<T, VEC>::load(y + c, v);
     Vec<T, VEC>::load(yw + c, w);
     Vec<float, VEC>::load(x + c, r);
 #pragma unroll
     for (int j = 0; j < VEC; ++j) {
-      r[j] += p.alpha * (v[j] * inv_y * w[j]);
+      r[j] += v[j] * inv_y * w[j];
       ss += r[j] * r[j];
-      if (c < step) kept[j] = r[j];
     }
     Vec<float, VEC>::store(x + c, r);
   }
   if (p.out == nullptr) return;
-  float inv_x = 1.f;
-  const T* nw = reinterpret_cast<const T*>(p.next_weight);
-  if (nw != nullptr) inv_x = 1.f / sqrtf(block_sum(ss, red[1]) / (float)p.cols + p.eps);
+  const float inv_x = nw == nullptr ? 1.f : 1.f / sqrtf(block_sum(ss, red[1]) / (float)p.cols + p.eps);
   T* out = reinterpret_cast<T*>(p.out) + (long long)blockIdx.x * p.ldo;
-  for (int c = tid * VEC; c < p.cols; c += step) {
-    float v[VEC];
-    if (c < step) {
-#pragma unroll
-      for (int j = 0; j < VEC; ++j) v[j] = kept[j];
-    } else {
-      Vec<float, VEC>::load(x + c, v);
-    }
+  auto emit = [&](int c, float (&v)[VEC]) {
     if (nw != nullptr) {
       float w[VEC];
       Vec<T, VEC>::load(nw + c, w);
@@ -86,6 +98,16 @@ __global__ void __launch_bounds__(1024) residual_norm_kernel(ResidualParams p) {
       for (int j = 0; j < VEC; ++j) v[j] = v[j] * inv_x * w[j];
     }
     Vec<T, VEC>::store(out + c, v);
+  };
+#pragma unroll
+  for (int k = 0; k < kKept; ++k) {
+    const int c = (k * blockDim.x + tid) * VEC;
+    if (c < p.cols) emit(c, sums[k]);
+  }
+  for (int c = (kKept * blockDim.x + tid) * VEC; c < p.cols; c += step) {
+    float v[VEC];
+    Vec<float, VEC>::load(x + c, v);
+    emit(c, v);
   }
 }
 
@@ -152,7 +174,7 @@ struct GatedNormParams {
 };
 
 template <typename T, int VEC>
-__global__ void __launch_bounds__(1024) gated_norm_kernel(GatedNormParams p) {
+__global__ void __launch_bounds__(512) gated_norm_kernel(GatedNormParams p) {
   __shared__ float red[32];
   chain_wait();
   chain_release();
@@ -160,31 +182,46 @@ __global__ void __launch_bounds__(1024) gated_norm_kernel(GatedNormParams p) {
   const T* x = reinterpret_cast<const T*>(p.x) + (long long)blockIdx.x * p.ldx;
   const T* gate = reinterpret_cast<const T*>(p.gate) + (long long)blockIdx.x * p.ldg;
   T* out = reinterpret_cast<T*>(p.out) + (long long)blockIdx.x * p.ldo;
-  float kept[VEC];
+  const T* weight = reinterpret_cast<const T*>(p.weight);
+  float xs[kKept][VEC], ws[kKept][VEC], gs[kKept][VEC];
   float ss = 0.f;
-  for (int c = tid * VEC; c < p.cols; c += step) {
+#pragma unroll
+  for (int k = 0; k < kKept; ++k) {
+    const int c = (k * blockDim.x + tid) * VEC;
+    if (c < p.cols) {
+      Vec<T, VEC>::load(x + c, xs[k]);
+      Vec<T, VEC>::load(weight + c, ws[k]);
+      Vec<T, VEC>::load(gate + c, gs[k]);
+    }
+  }
+#pragma unroll
+  for (int k = 0; k < kKept; ++k)
+    if ((k * (int)blockDim.x + tid) * VEC < p.cols)
+#pragma unroll
+      for (int j = 0; j < VEC; ++j) ss += xs[k][j] * xs[k][j];
+  for (int c = (kKept * blockDim.x + tid) * VEC; c < p.cols; c += step) {
     float v[VEC];
     Vec<T, VEC>::load(x + c, v);
 #pragma unroll
-    for (int j = 0; j < VEC; ++j) {
-      ss += v[j] * v[j];
-      if (c < step) kept[j] = v[j];
-    }
+    for (int j = 0; j < VEC; ++j) ss += v[j] * v[j];
   }
   const float inv = 1.f / sqrtf(block_sum(ss, red) / (float)p.cols + p.eps);
-  for (int c = tid * VEC; c < p.cols; c += step) {
-    float v[VEC], w[VEC], g[VEC];
-    if (c < step) {
+  auto emit = [&](int c, float (&v)[VEC], const float (&w)[VEC], const float (&g)[VEC]) {
 #pragma unroll
-      for (int j = 0; j < VEC; ++j) v[j] = kept[j];
-    } else {
-      Vec<T, VEC>::load(x + c, v);
-    }
-    Vec<T, VEC>::load(reinterpret_cast<const T*>(p.weight) + c, w);
-    Vec<T, VEC>::load(gate + c, g);
-#pragma unroll
-    for (int j = 0; j < VEC; ++j) v[j] = v[j] * inv * w[j] / (1.f + expf(-g[j]));
+    for (int j = 0; j < VEC; ++j) v[j] = __fdividef(v[j] * inv * w[j], 1.f + expf(-g[j]));
     Vec<T, VEC>::store(out + c, v);
+  };
+#pragma unroll
+  for (int k = 0; k < kKept; ++k) {
+    const int c = (k * blockDim.x + tid) * VEC;
+    if (c < p.cols) emit(c, xs[k], ws[k], gs[k]);
+  }
+  for (int c = (kKept * blockDim.x + tid) * VEC; c < p.cols; c += step) {
+    float v[VEC], w[VEC], g[VEC];
+    Vec<T, VEC>::load(x + c, v);
+    Vec<T, VEC>::load(weight + c, w);
+    Vec<T, VEC>::load(gate + c, g);
+    emit(c, v, w, g);
   }
 }
 
@@ -197,8 +234,9 @@ __global__ void softcap_kernel(float* logits, long long count, float cap) {
 }
 
 int row_threads(int cols, bool vec) {
-  const int threads = ((vec ? cols / 8 : cols) + 31) / 32 * 32;
-  return threads > 1024 ? 1024 : threads;
+  const int groups = vec ? cols / 8 : cols;
+  const int threads = ((groups + kKept - 1) / kKept + 31) / 32 * 32;
+  return threads > 512 ? 512 : threads;
 }
 
 // One CTA per row, in the vector width the rows allow.

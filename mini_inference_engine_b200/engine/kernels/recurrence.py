@@ -37,11 +37,12 @@ class StateBuffer:
 
 def segment_tokens(max_query_len: int, lanes: int, sm_count: int = 148) -> int:
     """Tokens per parallel segment of a packed chunk, 0 for one segment per request.  ``lanes`` is how many CTAs run
-    without cutting; requests are cut until the GPU has about two CTAs per SM to run, in pieces of at least 256."""
+    without cutting; requests are cut until the GPU has about one CTA per SM to run, in pieces of at least 256 (the
+    pieces but the last are gone over twice)."""
 
-    if max_query_len <= 256 or lanes >= sm_count:
+    if max_query_len <= 256 or 2 * lanes > sm_count:
         return 0
-    pieces = -(-2 * sm_count // max(lanes, 1))
+    pieces = sm_count // max(lanes, 1)
     length = -(-max_query_len // pieces)
     return max(256, -(-length // TILE) * TILE)
 
@@ -53,7 +54,7 @@ def outer_recurrence(rows, out, decay, state, slots, positions, *, heads: int, d
     tokens, requests = int(rows.shape[0]), 0 if cu_seqlens is None else int(cu_seqlens.shape[0]) - 1
     length, carry = 0, None
     if cu_seqlens is not None and _lib.load().mie_outer_recurrence_chunked(dim, value_dim, _lib.DTYPE_CODES[rows.dtype]):
-        length = segment_tokens(max_query_len, requests * heads * -(-value_dim // 64))
+        length = segment_tokens(max_query_len, requests * heads * -(-value_dim // 128))
         if length and max_query_len > length:
             carry = torch.empty((tokens // length + requests) * heads * dim * value_dim, dtype=torch.float32,
                                 device=rows.device)
