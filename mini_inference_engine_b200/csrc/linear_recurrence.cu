@@ -17,7 +17,22 @@
 namespace mie {
 namespace {
 
-__device__ __forceinline__ float silu(float v) { return __fdividef(v, 1.f + expf(-v)); }
+// 2^x and 1 / x on the special-function unit (about 22 bits).
+__device__ __forceinline__ float exp2_unit(float x) {
+  float y;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+__device__ __forceinline__ float reciprocal_unit(float x) {
+  float y;
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
+  return y;
+}
+// 1 + e^-v, the denominator of sigmoid(v); v bounded from below so that a product of two stays finite.
+__device__ __forceinline__ float sigmoid_denominator(float v) {
+  return 1.f + exp2_unit(fminf(v * -1.4426950408889634f, 60.f));
+}
+__device__ __forceinline__ float silu(float v) { return v * reciprocal_unit(1.f + exp2_unit(v * -1.4426950408889634f)); }
 
 struct Slots {
   float* state;
@@ -225,14 +240,6 @@ __device__ __forceinline__ uint32_t swizzled(int row, int unit) { return row * 1
 
 __device__ __forceinline__ uint32_t pack_bf16(float lo, float hi) { return Mma16816<__nv_bfloat16>::pack(lo, hi); }
 
-// silu of activations that are rounded to bf16 next.
-__device__ __forceinline__ float silu_rounded(float v) {
-  float e, r;
-  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(v * -1.4426950408889634f));
-  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.f + e));
-  return v * r;
-}
-
 // 16 bytes global -> shared, or zeros.
 __device__ __forceinline__ void copy_async16(uint32_t dst, const void* src, bool live) {
   asm volatile("cp.async.cg.shared.global [%0], [%1], 16, %2;" ::"r"(dst), "l"(src), "r"(live ? 16 : 0) : "memory");
@@ -327,7 +334,7 @@ __global__ void __launch_bounds__(256 * VD, KD + VD == 2 ? 2 : 1) outer_chunk_ke
     auto unpack = [&](float (&v)[8]) {
       Vec<T, 8>::load(reinterpret_cast<const T*>(staged), v);
 #pragma unroll
-      for (int j = 0; j < 8; ++j) v[j] = silu_rounded(v[j]);
+      for (int j = 0; j < 8; ++j) v[j] = silu(v[j]);
       staged += kThreads * 16;
     };
     // q and k through silu; rows past the segment and dims past the head are zero.
@@ -581,11 +588,10 @@ struct AverageParams {
   float* carry;  // [segments][2][width], null: every request is one segment
 };
 
-// keep = 1 - z, add = z * candidate.  The two sigmoids share one reciprocal; their exponents are bounded so that the
-// product of the denominators stays finite (a sigmoid below 1e-17 is 1e-17).
+// keep = 1 - z, add = z * candidate.  The two sigmoids share one reciprocal.
 __device__ __forceinline__ void average_gates(float a, float u, float* keep, float* add) {
-  const float da = 1.f + expf(fminf(-a, 40.f)), du = 1.f + expf(fminf(-u, 40.f));
-  const float inv = __fdividef(1.f, da * du);
+  const float da = sigmoid_denominator(a), du = sigmoid_denominator(u);
+  const float inv = reciprocal_unit(da * du);
   const float gate = inv * du;
   *keep = 1.f - gate;
   *add = gate * (u >= 0.f ? u + 0.5f : inv * da);

@@ -152,4 +152,11 @@ __host__ __device__ constexpr uint32_t instr_desc_f16(int bn, int ab_format, int
          ((uint32_t)b_mn_major << 16) | ((uint32_t)(bn >> 3) << 17) | ((uint32_t)(kUmmaM >> 4) << 24);
 }
 
+// The same for M = 64 or 128 rows, bf16 operands, A and B each K-major (0) or MN-major (1).  With M = 64 row r of D
+// is tensor-memory lane (r / 16) * 32 + r % 16.
+__host__ __device__ constexpr uint32_t instr_desc_bf16(int m, int n, int a_mn_major, int b_mn_major) {
+  return (1u << 4) | (1u << 7) | (1u << 10) | ((uint32_t)a_mn_major << 15) | ((uint32_t)b_mn_major << 16) |
+         ((uint32_t)(n >> 3) << 17) | ((uint32_t)(m >> 4) << 24);
+}
+
 }  // namespace mie

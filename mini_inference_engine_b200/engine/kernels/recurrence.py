@@ -72,7 +72,7 @@ def gated_average(rows, out, z_bias, u_bias, state, slots, positions, *, width: 
     tokens, requests = int(rows.shape[0]), 0 if cu_seqlens is None else int(cu_seqlens.shape[0]) - 1
     length, carry = 0, None
     if cu_seqlens is not None and max_query_len > TILE:
-        length = TILE
+        length = TILE if tokens * width >= 64 * 512 * 296 else TILE // 2  # shorter pieces when they are few
         carry = torch.empty((tokens // length + requests) * 2 * width, dtype=torch.float32, device=rows.device)
     _lib.check(_lib.load().mie_gated_average(
         _lib.ptr(rows), rows.stride(0), _lib.ptr(z_bias), _lib.ptr(u_bias), _lib.ptr(out), out.stride(0),
