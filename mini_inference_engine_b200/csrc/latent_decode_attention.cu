@@ -3,16 +3,19 @@
 // once for both products and for all heads.
 //
 // One persistent CTA per SM walks (request, chunk, up to 32 heads) items of the shared split-KV plan in a fixed order.
-// The products run on tcgen05 with the cached rows as the A operand, so that their cost follows the number of heads:
-//   S = K Q^T      64 keys x heads, K-major rows of the stage, into one of two TMEM buffers (lane = key)
-//   softmax        a thread per key: common running maximum of every head (moved only when it grows by more than 2^8),
-//                  exp2, the weights as a rounded bf16 part beside its remainder in one shared-memory row per key
-//   O += V^T P     128 value dims x (2 x heads) per group, the same stage read MN-major; rounded parts and remainders
-//                  accumulate in neighbouring TMEM columns (lane = dim) and are added at the end
-// Warp roles: 4 softmax / epilogue warps, 1 TMA producer (16-token slabs of pages into a ring of 64-token stages,
-// 128-byte swizzle, no multicast) that runs ahead across items, 1 MMA issuer that owns the TMEM allocation.  Every wait
-// is bounded and reports MIE_STATUS_WAIT_TIMEOUT.  Scores, weights, sums and O are fp32.  The sink opens the running
-// maximum and the denominator of a request's first chunk; partials are merged by merge_rows_kernel.
+// Warp roles: 8 score warps, 1 TMA producer (16-token slabs of pages into a ring of 64-token stages, 128-byte swizzle,
+// no multicast) that runs ahead across items, 1 tcgen05 issuer that owns the TMEM allocation.  Per stage:
+//   S = K Q^T    mma.sync; a warp has 16 heads, 16 * MT keys and every other 16 dims (with one 16-head tile its Q
+//                fragments stay in registers); the two warps that share keys swap halves of their sums
+//   softmax      row maxima meet in shared memory; the common reference maximum moves only when a head's grows by more
+//                than 2^8; the weights go to shared memory as a rounded bf16 part and its remainder, one row per head each
+//   O += V^T P   tcgen05, A = 128 value dims of the stage read MN-major, B = the weight rows: rounded parts and
+//                remainders accumulate in neighbouring TMEM columns (lane = dim) and are added at the end.  It runs while
+//                the score warps are at the next stage
+// (tcgen05 streams A at one row per cycle whatever the number of heads, mma.sync pays per 16 heads: for up to 32 heads
+// the first product is cheaper on mma.sync and the second on tcgen05, and the two overlap.)  Every wait is bounded and
+// reports MIE_STATUS_WAIT_TIMEOUT.  Scores, weights, sums and O are fp32.  The sink opens the running maximum and the
+// denominator of a request's first chunk; partials are merged by merge_rows_kernel.
 #include "decode_attention.cuh"
 #include "umma.cuh"
 
@@ -27,8 +30,8 @@ bool pages_fit_slab_map(const mie_view4_t& v, int block_size, int dim);
 namespace {
 
 constexpr int kStageTokens = 64;
-constexpr int kSoftmaxWarps = 4;
-constexpr int kLatentThreads = (kSoftmaxWarps + 2) * 32;
+constexpr int kScoreWarps = 8;
+constexpr int kLatentThreads = (kScoreWarps + 2) * 32;
 constexpr int kMaxKeyBoxes = 10;
 constexpr int kMaxValueDims = 512;
 constexpr int kItemHeads = 32;               // heads one work item covers at most
@@ -49,36 +52,34 @@ struct LatentParams {
   int* status;
 };
 
-// Shared memory: ring of stages | Q [box][head][64] | P, two buffers of [key][rounded heads | remainders] | warp maxima
-// and sums [warp][head] | barriers.
+// Shared memory: ring of stages | Q [box][head][64] | P, two buffers of [rounded heads | remainders][64 keys] | swapped
+// sums | two [head][key group] of maxima, one of denominators | factors per head | barriers.
 struct LatentLayout {
-  int stage, q, p, maxima, bars, total;
+  int stage, q, p, p_bytes, swap, maxima, sums, factors, bars, total;
 };
-constexpr int kPBytes = kStageTokens * 128;
-__host__ __device__ inline LatentLayout latent_layout(int key_boxes, int ring, int heads) {
+__host__ __device__ inline LatentLayout latent_layout(int key_boxes, int ring, int tiles) {
   LatentLayout l;
+  const int heads = tiles * 16;
   l.stage = key_boxes * kStageTokens * 128;
   l.q = ring * l.stage;
   l.p = l.q + key_boxes * heads * 128;
-  l.maxima = l.p + 2 * kPBytes;
-  l.bars = l.maxima + 2 * kSoftmaxWarps * heads * 4;
+  l.p_bytes = 2 * heads * 128;
+  l.swap = l.p + 2 * l.p_bytes;
+  l.maxima = l.swap + kScoreWarps * 32 * tiles * 16;
+  l.sums = l.maxima + 2 * heads * 8 * 4;
+  l.factors = l.sums + heads * 8 * 4;
+  l.bars = l.factors + heads * 4;
   l.total = l.bars + 256;
   return l;
 }
 constexpr int kMaxRing = 4;
-enum LatentBar { kFull = 0, kEmpty = kMaxRing, kQFull = 2 * kMaxRing, kSFull, kPFull = kSFull + 2, kPvDone = kPFull + 2,
-                 kOFree = kPvDone + 2, kLatentBars };
+enum LatentBar { kFull = 0, kEmpty = kMaxRing, kPFull = 2 * kMaxRing, kPvDone = kPFull + 2, kOFree = kPvDone + 2,
+                 kLatentBars };
 
-__device__ __forceinline__ void softmax_sync() { asm volatile("bar.sync 1, 128;" ::: "memory"); }
+__device__ __forceinline__ void score_sync() { asm volatile("bar.sync 1, 256;" ::: "memory"); }
 __device__ __forceinline__ float ex2_approx(float x) {  // -inf gives +0
   float y;
   asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(y) : "f"(x));
-  return y;
-}
-// Largest value of the warp in one instruction (warp-wide redux on fp32).
-__device__ __forceinline__ float warp_most(float x) {
-  float y;
-  asm volatile("redux.sync.max.f32 %0, %1, 0xffffffff;" : "=f"(y) : "f"(x));
   return y;
 }
 // Columns of this thread's TMEM lane.
@@ -102,40 +103,41 @@ struct LatentItem {
   }
 };
 
-template <int HN>  // heads per item, 16 or 32
+// MT: 16-head tiles per item.  BOXES: 64-dim boxes of the key (the last one zero-filled past the key's size).
+template <int MT, int BOXES>
 __global__ void __launch_bounds__(kLatentThreads, 1)
     latent_decode_kernel(const __grid_constant__ CUtensorMap map, const LatentParams p) {
   using T = __nv_bfloat16;
+  using Mma = Mma16816<T>;
+  constexpr int HN = MT * 16;
   extern __shared__ uint8_t latent_smem_raw[];
   uint8_t* smem = reinterpret_cast<uint8_t*>(align_up((long long)reinterpret_cast<uintptr_t>(latent_smem_raw), 1024));
-  const LatentLayout at = latent_layout(p.key_boxes, p.ring, HN);
+  const LatentLayout at = latent_layout(BOXES, p.ring, MT);
   uint64_t* bars = reinterpret_cast<uint64_t*>(smem + at.bars);
   uint32_t* tmem_slot = reinterpret_cast<uint32_t*>(bars + kLatentBars);
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
-  constexpr uint32_t kTmemCols = 512;
+  constexpr uint32_t kTmemCols = kMaxValueDims / 128 * 2 * HN;  // 2 HN columns per group of 128 value dims
   if (threadIdx.x == 0) {
     for (int s = 0; s < p.ring; ++s) {
       mbar_init(&bars[kFull + s], 1);
       mbar_init(&bars[kEmpty + s], 1);
     }
-    mbar_init(&bars[kQFull], kSoftmaxWarps * 32);
-    mbar_init(&bars[kOFree], kSoftmaxWarps * 32);
+    mbar_init(&bars[kOFree], kScoreWarps * 32);
     for (int b = 0; b < 2; ++b) {
-      mbar_init(&bars[kSFull + b], 1);
-      mbar_init(&bars[kPFull + b], kSoftmaxWarps * 32);
+      mbar_init(&bars[kPFull + b], kScoreWarps * 32);
       mbar_init(&bars[kPvDone + b], 1);
     }
     mbar_fence_init();
     tma_prefetch_desc(&map);
   }
-  if (warp == kSoftmaxWarps + 1) {
+  if (warp == kScoreWarps + 1) {
     tmem_alloc(tmem_slot, kTmemCols);
     tmem_relinquish();
   }
   tc_fence_before();
   __syncthreads();
   tc_fence_after();
-  const uint32_t tmem_s = *tmem_slot, tmem_o = *tmem_slot + 2 * HN;  // S: 2 x HN columns, O: 2 HN columns per group
+  const uint32_t tmem_o = *tmem_slot;
   chain_wait();
   chain_release();
 
@@ -155,10 +157,10 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
     return it;
   };
   // Byte distance between 8-token groups and between 64-dim groups of a stage.
-  const int tok_group = p.slab ? p.key_boxes * 1024 : 1024, dim_group = p.slab ? 1024 : kStageTokens * 128;
+  const int tok_group = p.slab ? BOXES * 1024 : 1024, dim_group = p.slab ? 1024 : kStageTokens * 128;
   const int value_groups = (p.vdim + 127) / 128;
 
-  if (warp == kSoftmaxWarps) {
+  if (warp == kScoreWarps) {
     // ---------------- TMA producer ----------------
     const uint64_t policy = l2_evict_first_policy();
     int fill = 0;  // stages filled so far
@@ -179,7 +181,7 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         if (lane == 0) {
           ok = mbar_wait_bounded(&bars[kEmpty + s], ((fill / p.ring) & 1u) ^ 1u);
           if (ok)
-            mbar_expect_tx(&bars[kFull + s], slabs * p.key_boxes * kBoxBytes);
+            mbar_expect_tx(&bars[kFull + s], slabs * BOXES * kBoxBytes);
           else
             raise_status(p.status, MIE_STATUS_WAIT_TIMEOUT);
         }
@@ -187,55 +189,42 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         if (ok && lane < slabs) {
           uint8_t* dst = smem + s * at.stage;
           if (p.slab) {
-            tma_load_5d_hint(dst + lane * p.key_boxes * kBoxBytes, &map, &bars[kFull + s], 0, 0, 0, slot / 8, page, policy);
+            tma_load_5d_hint(dst + lane * BOXES * kBoxBytes, &map, &bars[kFull + s], 0, 0, 0, slot / 8, page, policy);
           } else {
-            for (int x = 0; x < p.key_boxes; ++x)
+            for (int x = 0; x < BOXES; ++x)
               tma_load_4d_hint(dst + x * dim_group + lane * kBoxBytes, &map, &bars[kFull + s], x * 64, slot, 0, page, policy);
           }
         }
         __syncwarp();
       }
     }
-  } else if (warp == kSoftmaxWarps + 1) {
-    // ---------------- MMA issuer ----------------
+  } else if (warp == kScoreWarps + 1) {
+    // ---------------- tcgen05 issuer ----------------
     if (lane == 0) {
-      constexpr uint32_t idesc_s = instr_desc_bf16(64, HN, 0, 0);        // A = K rows, B = Q rows, both K-major
-      constexpr uint32_t idesc_o = instr_desc_bf16(128, 2 * HN, 1, 1);   // A = V^T, B = P, both MN-major
-      const int k_steps = (p.dim + 15) / 16;
-      const uint32_t q_addr = smem_u32(smem + at.q), p_addr = smem_u32(smem + at.p);
+      constexpr uint32_t idesc = instr_desc_bf16(128, 2 * HN, 1, 0);  // A = V^T, MN-major; B = weight rows, K-major
+      // Descriptor addresses count 16-byte units: every product's operands are a base plus small increments.
+      const uint64_t slab_step = (2 * tok_group) >> 4, group_step = (2 * dim_group) >> 4;
       int tile = 0, items = 0;  // stages and items so far
       bool ok = true;
       for (int number = blockIdx.x; number < total_items && ok; number += gridDim.x, ++items) {
         const LatentItem it = item_of(number);
-        const int tiles = (int)((it.end - it.begin + kStageTokens - 1) / kStageTokens);
-        ok = mbar_wait_bounded(&bars[kQFull], items & 1u);
-        // S(j) overwrites the buffer whose P(j - 2) was waited for before P V(j - 2) was issued.
-        auto issue_s = [&](int j) {
-          const int s = j % p.ring, b = j & 1;
-          if (!mbar_wait_bounded(&bars[kFull + s], (j / p.ring) & 1u)) return false;
-          tc_fence_after();
-          const uint32_t k_addr = smem_u32(smem + s * at.stage);
-          for (int ks = 0; ks < k_steps; ++ks)
-            umma_f16(tmem_s + b * HN, smem_desc_k128(k_addr + (ks >> 2) * dim_group + (ks & 3) * 32, tok_group),
-                     smem_desc_k128(q_addr + (ks >> 2) * (HN * 128) + (ks & 3) * 32), idesc_s, ks > 0 ? 1u : 0u);
-          umma_commit(&bars[kSFull + b]);
-          return true;
-        };
-        if (ok) ok = issue_s(tile);
-        for (int j = 0; j < tiles && ok; ++j, ++tile) {
+        for (long long tok0 = it.begin; tok0 < it.end && ok; tok0 += kStageTokens, ++tile) {
           const int s = tile % p.ring, b = tile & 1;
-          if (j + 1 < tiles) ok = issue_s(tile + 1);
-          if (ok) ok = mbar_wait_bounded(&bars[kPFull + b], (tile >> 1) & 1u);
-          if (ok && j == 0 && items > 0) ok = mbar_wait_bounded(&bars[kOFree], (items - 1) & 1u);  // O has been read
+          ok = mbar_wait_bounded(&bars[kPFull + b], (tile >> 1) & 1u) &&
+               mbar_wait_bounded(&bars[kFull + s], (tile / p.ring) & 1u) &&
+               (tok0 > it.begin || items == 0 || mbar_wait_bounded(&bars[kOFree], (items - 1) & 1u));  // O has been read
           if (!ok) break;
           tc_fence_after();
-          const uint32_t v_addr = smem_u32(smem + s * at.stage);
-          const int slabs = (it.valid(it.begin + (long long)j * kStageTokens) + kTileTokens - 1) / kTileTokens;
+          uint64_t values = smem_desc_mn128(smem_u32(smem + s * at.stage), dim_group, tok_group);
+          uint64_t weights = smem_desc_k128(smem_u32(smem + at.p + b * at.p_bytes));
+          const int slabs = (it.valid(tok0) + kTileTokens - 1) / kTileTokens;
           for (int kt = 0; kt < slabs; ++kt) {
-            const uint64_t weights = smem_desc_mn128(p_addr + b * kPBytes + kt * 2048, 1024, 1024);
-            for (int d = 0; d < value_groups; ++d)
-              umma_f16(tmem_o + d * 2 * HN, smem_desc_mn128(v_addr + 2 * d * dim_group + kt * 2 * tok_group, dim_group, tok_group),
-                       weights, idesc_o, j > 0 || kt > 0 ? 1u : 0u);
+#pragma unroll
+            for (int d = 0; d < kMaxValueDims / 128; ++d)
+              if (d < value_groups)
+                umma_f16(tmem_o + d * 2 * HN, values + d * group_step, weights, idesc, tok0 > it.begin || kt > 0 ? 1u : 0u);
+            values += slab_step;
+            weights += 2;
           }
           umma_commit(&bars[kEmpty + s]);   // the stage is free once these MMAs have read it
           umma_commit(&bars[kPvDone + b]);  // O includes this stage
@@ -244,130 +233,215 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
       if (!ok) raise_status(p.status, MIE_STATUS_WAIT_TIMEOUT);
     }
   } else {
-    // ---------------- Softmax and epilogue: thread = key of a stage, then thread = value dim ----------------
-    const uint32_t lane_addr = (uint32_t)(warp * 32) << 16;
-    const int key = warp * 16 + lane;  // lanes 0 ... 15
-    float* maxima = reinterpret_cast<float*>(smem + at.maxima);  // [warp][head], double-buffered by stage parity
-    bool ok = true;
-    auto load_q = [&](const LatentItem& it) {
-      for (int i = threadIdx.x; i < HN * p.key_boxes * 8; i += kSoftmaxWarps * 32) {
-        const int r = i / (p.key_boxes * 8), u = i % (p.key_boxes * 8), head = it.group * HN + r;
+    // ---------------- scores, softmax, epilogue ----------------
+    const int g = lane >> 2, t = lane & 3;
+    // S: warp = (16-head tile mt_s, every other 16-dim step from k_half on, 16 * MT keys of pair kp); after the swap it
+    // owns kKeys of them, group kg.
+    constexpr int kKeys = 8 * MT;
+    constexpr int kKeyGroups = kStageTokens / kKeys;
+    constexpr int kSteps = BOXES * 2;  // 16-dim steps of one half
+    constexpr int kAhead = 3;          // steps whose operands are loaded before they are used
+    constexpr bool kHoldQ = MT == 1;
+    const int mt_s = warp % MT, k_half = warp / MT % 2, kp = warp / (2 * MT);
+    const int kg = 2 * kp + k_half;
+    const uint32_t q_at = smem_u32(smem + at.q);
+    float* swap = reinterpret_cast<float*>(smem + at.swap);
+    float* maxima = reinterpret_cast<float*>(smem + at.maxima);    // [stage parity][head][key group]
+    float* sums = reinterpret_cast<float*>(smem + at.sums);        // [head][key group]
+    float* factors = reinterpret_cast<float*>(smem + at.factors);  // [head]
+    const int a_row = (lane & 7) + ((lane >> 3) & 1) * 8, a_sel = (lane >> 4) & 1;
+    const int k_row = (lane & 7) + ((lane >> 4) & 1) * 8, k_sel = (lane >> 3) & 1;  // sixteen keys x 16 dims per load
+    const uint32_t lane_addr = (uint32_t)((warp & 3) * 32) << 16;                   // O: TMEM lanes of this warp
+    auto fetch_q = [&](const LatentItem& it) {
+      for (int i = threadIdx.x; i < HN * BOXES * 8; i += kScoreWarps * 32) {
+        const int r = i / (BOXES * 8), u = i % (BOXES * 8), head = it.group * HN + r;
         uint4 v = make_uint4(0, 0, 0, 0);
         if (head < p.heads && u * 8 < p.dim)
           v = *reinterpret_cast<const uint4*>(p.q + (it.request * p.q_row + head * p.q_head + u * 8) * 2);
         *reinterpret_cast<uint4*>(smem + at.q + (u >> 3) * (HN * 128) + r * 128 + (((u & 7) ^ (r & 7)) << 4)) = v;
       }
-      fence_proxy_async_smem();
-      mbar_arrive(&bars[kQFull]);
     };
-    LatentItem it;
     int tile = 0;
+    bool ok = true;  // a failed wait skips later waits, never a barrier
+    LatentItem it;
     if ((int)blockIdx.x < total_items) {
       it = item_of(blockIdx.x);
-      load_q(it);
+      fetch_q(it);
     }
     for (int number = blockIdx.x; number < total_items; number += gridDim.x) {
       const int head0 = it.group * HN;
-      float m[HN], l[HN];  // reference maximum (log2 units, the same in every thread); this key's share of the denominator
+      score_sync();  // Q is there
+      auto load_q = [&](int ks, uint32_t (&a)[4]) {
+        ldmatrix_x4(a[0], a[1], a[2], a[3], q_at + (ks >> 2) * (HN * 128) + (mt_s * 16 + a_row) * 128 +
+                                                ((((ks & 3) * 2 + a_sel) ^ (a_row & 7)) << 4));
+      };
+      uint32_t held[kHoldQ ? kSteps : 1][4];
+      if (kHoldQ) {
 #pragma unroll
-      for (int h = 0; h < HN; ++h) {
-        m[h] = -INFINITY;
-        l[h] = 0.f;
-        if (p.sinks != nullptr && it.chunk == 0) {
-          m[h] = head0 + h < p.heads ? p.sinks[head0 + h] * kLog2e : 0.f;
-          if (threadIdx.x == 0) l[h] = 1.f;
-        }
+        for (int i = 0; i < kSteps; ++i) load_q(2 * i + k_half, held[kHoldQ ? i : 0]);
       }
-      bool first = true;
-      for (long long tok0 = it.begin; tok0 < it.end; tok0 += kStageTokens, ++tile) {
-        const int b = tile & 1, valid = it.valid(tok0);
-        if (ok && !mbar_wait_bounded(&bars[kSFull + b], (tile >> 1) & 1u)) ok = false;
-        tc_fence_after();
-        float s[HN];
-        tmem_load<HN>(tmem_s + b * HN + lane_addr, s);
-        const bool seen = lane < 16 && key < valid && tok0 + key >= it.first_seen;
-        float* mine = maxima + b * kSoftmaxWarps * HN;
-        float top = -INFINITY;
+      // Reference maximum (log2 units) of rows g, g + 8 of every 16-head tile; the denominators of this thread's own
+      // rows over its own keys.
+      float m[MT][2], l[2] = {0.f, 0.f};
 #pragma unroll
-        for (int h = 0; h < HN; ++h) {
-          s[h] = seen ? s[h] * p.scale_log2 : -INFINITY;
-          const float most = warp_most(s[h]);
-          if (lane == h) top = most;
+      for (int i = 0; i < MT; ++i)
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          m[i][e] = -INFINITY;
+          if (p.sinks != nullptr && it.chunk == 0) {
+            const int head = head0 + i * 16 + g + e * 8;
+            m[i][e] = head < p.heads ? p.sinks[head] * kLog2e : 0.f;
+            if (i == mt_s && kg == 0 && t == 0) l[e] = 1.f;
+          }
         }
-        if (lane < HN) mine[warp * HN + lane] = top;
+      for (long long tok0 = it.begin; tok0 < it.end; tok0 += kStageTokens, ++tile) {
+        const int s = tile % p.ring, b = tile & 1, valid = it.valid(tok0);
+        if (ok && !mbar_wait_bounded(&bars[kFull + s], (tile / p.ring) & 1u)) ok = false;
+        const uint32_t stage = smem_u32(smem + s * at.stage);
+        // Half sums of S for 16 heads x 16 * MT keys.
+        float part[2 * MT][4];
+#pragma unroll
+        for (int n = 0; n < 2 * MT; ++n) part[n][0] = part[n][1] = part[n][2] = part[n][3] = 0.f;
+        uint32_t keys[kAhead][MT][4], rows[kHoldQ ? 1 : kAhead][4];
+        auto load_keys = [&](int i) {
+          const int ks = 2 * i + k_half;
+          if (!kHoldQ) load_q(ks, rows[kHoldQ ? 0 : i % kAhead]);
+#pragma unroll
+          for (int np = 0; np < MT; ++np) {
+            const int key_row = (kp * MT + np) * 16 + k_row;
+            uint32_t(&k)[4] = keys[i % kAhead][np];
+            ldmatrix_x4(k[0], k[1], k[2], k[3],
+                        stage + (key_row >> 3) * tok_group + (key_row & 7) * 128 + (ks >> 2) * dim_group +
+                            ((((ks & 3) * 2 + k_sel) ^ (key_row & 7)) << 4));
+          }
+        };
+#pragma unroll
+        for (int i = 0; i < kAhead - 1 && i < kSteps; ++i) load_keys(i);
+#pragma unroll
+        for (int i = 0; i < kSteps; ++i) {
+          if (i + kAhead - 1 < kSteps) load_keys(i + kAhead - 1);
+          const uint32_t(&q)[4] = kHoldQ ? held[i % (kHoldQ ? kSteps : 1)] : rows[kHoldQ ? 0 : i % kAhead];
+#pragma unroll
+          for (int np = 0; np < MT; ++np) {
+            const uint32_t(&k)[4] = keys[i % kAhead][np];
+            Mma::run(part[2 * np], q[0], q[1], q[2], q[3], k[0], k[1]);
+            Mma::run(part[2 * np + 1], q[0], q[1], q[2], q[3], k[2], k[3]);
+          }
+        }
+        // Swap with the warp that has the other dims: each of the pair keeps half of the keys.
+        float sa[MT][4];
+#pragma unroll
+        for (int n = 0; n < MT; ++n) {
+          float4 give;
+          if (k_half == 0) {
+            give = make_float4(part[MT + n][0], part[MT + n][1], part[MT + n][2], part[MT + n][3]);
+            sa[n][0] = part[n][0], sa[n][1] = part[n][1], sa[n][2] = part[n][2], sa[n][3] = part[n][3];
+          } else {
+            give = make_float4(part[n][0], part[n][1], part[n][2], part[n][3]);
+            sa[n][0] = part[MT + n][0], sa[n][1] = part[MT + n][1], sa[n][2] = part[MT + n][2], sa[n][3] = part[MT + n][3];
+          }
+          *reinterpret_cast<float4*>(swap + ((warp * MT + n) * 32 + lane) * 4) = give;
+        }
+        asm volatile("bar.sync %0, 64;" ::"r"(2 + kp * MT + mt_s) : "memory");
+        float mx[2] = {-INFINITY, -INFINITY};
+#pragma unroll
+        for (int n = 0; n < MT; ++n) {
+          const int other = k_half == 0 ? warp + MT : warp - MT;
+          const float4 v = *reinterpret_cast<const float4*>(swap + ((other * MT + n) * 32 + lane) * 4);
+          sa[n][0] += v.x, sa[n][1] += v.y, sa[n][2] += v.z, sa[n][3] += v.w;
+#pragma unroll
+          for (int e = 0; e < 4; ++e) {
+            const int key = kg * kKeys + n * 8 + 2 * t + (e & 1);
+            sa[n][e] = key >= valid || tok0 + key < it.first_seen ? -INFINITY : sa[n][e] * p.scale_log2;
+            mx[e >> 1] = fmaxf(mx[e >> 1], sa[n][e]);
+          }
+        }
+#pragma unroll
+        for (int e = 0; e < 2; ++e) {
+          mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 1));
+          mx[e] = fmaxf(mx[e], __shfl_xor_sync(0xffffffffu, mx[e], 2));
+          if (t == 0) maxima[(b * HN + mt_s * 16 + g + e * 8) * 8 + kg] = mx[e];
+        }
         if (valid % kTileTokens != 0) {
           // Rows of the last slab past the read length may hold anything (even NaN bits): zero them so that 0 * V stays 0.
-          const int s0 = tile % p.ring, end = (valid + kTileTokens - 1) / kTileTokens * kTileTokens;
-          for (int i = threadIdx.x; i < (end - valid) * p.key_boxes * 8; i += kSoftmaxWarps * 32) {
-            const int row = valid + i / (p.key_boxes * 8), u = i % (p.key_boxes * 8);
-            *reinterpret_cast<uint4*>(smem + s0 * at.stage + (row >> 3) * tok_group + (u >> 3) * dim_group +
+          const int end = (valid + kTileTokens - 1) / kTileTokens * kTileTokens;
+          for (int i = threadIdx.x; i < (end - valid) * BOXES * 8; i += kScoreWarps * 32) {
+            const int row = valid + i / (BOXES * 8), u = i % (BOXES * 8);
+            *reinterpret_cast<uint4*>(smem + s * at.stage + (row >> 3) * tok_group + (u >> 3) * dim_group +
                                       (row & 7) * 128 + (u & 7) * 16) = make_uint4(0, 0, 0, 0);
           }
         }
-        softmax_sync();
-        bool grow = false;  // the same in every thread
-        float next[HN];
+        score_sync();
+        // Reference maxima; every warp looks at every head, so all decide alike whether any of them moves.
+        float next[MT][2];
+        bool grow = false;
 #pragma unroll
-        for (int h = 0; h < HN; h += 4) {
-          float4 a = *reinterpret_cast<const float4*>(mine + h);
+        for (int i = 0; i < MT; ++i)
 #pragma unroll
-          for (int w = 1; w < kSoftmaxWarps; ++w) {
-            const float4 c = *reinterpret_cast<const float4*>(mine + w * HN + h);
-            a.x = fmaxf(a.x, c.x), a.y = fmaxf(a.y, c.y), a.z = fmaxf(a.z, c.z), a.w = fmaxf(a.w, c.w);
+          for (int e = 0; e < 2; ++e) {
+            const float4* row = reinterpret_cast<const float4*>(maxima + (b * HN + i * 16 + g + e * 8) * 8);
+            const float4 a = row[0];
+            float top = fmaxf(fmaxf(a.x, a.y), fmaxf(a.z, a.w));
+            if (kKeyGroups > 4) {
+              const float4 c = row[1];
+              top = fmaxf(top, fmaxf(fmaxf(c.x, c.y), fmaxf(c.z, c.w)));
+            }
+            // Finite: every stage holds a visible token.
+            next[i][e] = top > m[i][e] + kRescaleThreshold ? top : m[i][e];
+            grow = grow || next[i][e] != m[i][e];
           }
-          next[h] = a.x, next[h + 1] = a.y, next[h + 2] = a.z, next[h + 3] = a.w;
-        }
-#pragma unroll
-        for (int h = 0; h < HN; ++h) {
-          // Every stage holds a visible token, so the maximum is finite.
-          if (next[h] <= m[h] + kRescaleThreshold) next[h] = m[h];
-          grow = grow || next[h] != m[h];
-        }
-        if (grow) {
-          if (!first) {
+        if (__any_sync(0xffffffffu, grow)) {
+          if (tok0 > it.begin) {
             // O must first hold every stage before this one; then its columns move to the new reference.
             if (ok && !mbar_wait_bounded(&bars[kPvDone + (b ^ 1)], ((tile - 1) >> 1) & 1u)) ok = false;
             tc_fence_after();
-            for (int d = 0; d < value_groups; ++d)
+            if (warp == 0 && t == 0) {
 #pragma unroll
-              for (int part = 0; part < 2; ++part) {
-                const uint32_t addr = tmem_o + d * 2 * HN + part * HN + lane_addr;
+              for (int i = 0; i < MT; ++i)
+#pragma unroll
+                for (int e = 0; e < 2; ++e) factors[i * 16 + g + e * 8] = ex2_approx(m[i][e] - next[i][e]);
+            }
+            score_sync();
+            for (int d = warp >> 2; d < value_groups; d += 2)
+#pragma unroll
+              for (int half = 0; half < 2; ++half) {
+                const uint32_t addr = tmem_o + d * 2 * HN + half * HN + lane_addr;
                 float v[HN];
                 tmem_load<HN>(addr, v);
 #pragma unroll
-                for (int h = 0; h < HN; ++h) v[h] *= ex2_approx(m[h] - next[h]);
+                for (int h = 0; h < HN; ++h) v[h] *= factors[h];
                 if constexpr (HN == 16)
                   tmem_st16(addr, *reinterpret_cast<const uint32_t(*)[16]>(&v));
                 else
                   tmem_st32(addr, *reinterpret_cast<const uint32_t(*)[32]>(&v));
               }
             tmem_st_wait();
+            score_sync();  // `factors` may be written again
           }
 #pragma unroll
-          for (int h = 0; h < HN; ++h) {
-            l[h] *= ex2_approx(m[h] - next[h]);  // 0 * 0 while nothing has been seen
-            m[h] = next[h];
-          }
+          for (int i = 0; i < MT; ++i)
+#pragma unroll
+            for (int e = 0; e < 2; ++e) {
+              if (i == mt_s) l[e] *= ex2_approx(m[i][e] - next[i][e]);
+              m[i][e] = next[i][e];
+            }
         }
-        first = false;
         // P(tile) goes where P(tile - 2) was.
         if (ok && tile >= 2 && !mbar_wait_bounded(&bars[kPvDone + b], ((tile - 2) >> 1) & 1u)) ok = false;
-        if (lane < 16) {
-          uint8_t* row = smem + at.p + b * kPBytes + key * 128;
 #pragma unroll
-          for (int h = 0; h < HN; h += 8) {
-            uint32_t high[4], low[4];
+        for (int n = 0; n < MT; ++n) {
+          const int key = kg * kKeys + n * 8 + 2 * t;
 #pragma unroll
-            for (int j = 0; j < 4; ++j) {
-              const float w0 = ex2_approx(s[h + 2 * j] - m[h + 2 * j]), w1 = ex2_approx(s[h + 2 * j + 1] - m[h + 2 * j + 1]);
-              l[h + 2 * j] += w0;
-              l[h + 2 * j + 1] += w1;
-              high[j] = Mma16816<T>::pack(w0, w1);
-              const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&high[j]));
-              low[j] = Mma16816<T>::pack(w0 - k.x, w1 - k.y);
-            }
-            *reinterpret_cast<uint4*>(row + (((h >> 3) ^ (key & 7)) << 4)) = make_uint4(high[0], high[1], high[2], high[3]);
-            *reinterpret_cast<uint4*>(row + ((((HN + h) >> 3) ^ (key & 7)) << 4)) = make_uint4(low[0], low[1], low[2], low[3]);
+          for (int e = 0; e < 2; ++e) {
+            const float ref = mt_s == 0 ? m[0][e] : m[MT - 1][e];
+            const float w0 = ex2_approx(sa[n][2 * e] - ref), w1 = ex2_approx(sa[n][2 * e + 1] - ref);
+            l[e] += w0 + w1;
+            const int row = mt_s * 16 + g + e * 8;
+            uint8_t* dst = smem + at.p + b * at.p_bytes + row * 128 + (((key >> 3) ^ (row & 7)) << 4) + (key & 7) * 2;
+            const uint32_t high = Mma::pack(w0, w1);
+            const float2 k = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&high));
+            *reinterpret_cast<uint32_t*>(dst) = high;
+            *reinterpret_cast<uint32_t*>(dst + HN * 128) = Mma::pack(w0 - k.x, w1 - k.y);
           }
         }
         fence_proxy_async_smem();
@@ -375,62 +449,61 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
         mbar_arrive(&bars[kPFull + b]);
       }
       const LatentItem done = it;
+      // Denominators: over the quad, then over the key groups.
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        l[e] += __shfl_xor_sync(0xffffffffu, l[e], 1);
+        l[e] += __shfl_xor_sync(0xffffffffu, l[e], 2);
+        if (t == 0) sums[(mt_s * 16 + g + e * 8) * 8 + kg] = l[e];
+      }
       if (number + (int)gridDim.x < total_items) {  // the next item's queries, while the last products run
         it = item_of(number + gridDim.x);
-        load_q(it);
+        fetch_q(it);
       }
-      // Denominators: over the warp, then over the warps.
-      float* sums = maxima + (tile & 1) * kSoftmaxWarps * HN;  // not the buffer the last stage's maxima are read from
-      float mine = 0.f;
+      score_sync();
+      const long long part0 = ((long long)p.sc.offsets[done.request] + done.chunk) * p.heads + head0;
+      if (warp == 0 && t == 0) {
 #pragma unroll
-      for (int h = 0; h < HN; ++h) {
-        const float total = warp_sum(l[h]);
-        if (lane == h) mine = total;
+        for (int i = 0; i < MT; ++i)
+#pragma unroll
+          for (int e = 0; e < 2; ++e) {
+            const int h = i * 16 + g + e * 8;
+            float total = 0.f;
+#pragma unroll
+            for (int k = 0; k < kKeyGroups; ++k) total += sums[h * 8 + k];
+            factors[h] = done.chunks == 1 ? 1.f / fmaxf(total, 1.17549435e-38f) : 1.f;
+            if (done.chunks > 1 && head0 + h < p.heads) {
+              p.sc.part_m[part0 + h] = m[i][e];
+              p.sc.part_l[part0 + h] = total;
+            }
+          }
       }
-      if (lane < HN) sums[warp * HN + lane] = mine;
-      softmax_sync();
       const int last = tile - 1;
       if (ok && !mbar_wait_bounded(&bars[kPvDone + (last & 1)], (last >> 1) & 1u)) ok = false;
       tc_fence_after();
-#pragma unroll
-      for (int h = 0; h < HN; ++h) {
-        float total = 0.f;
-#pragma unroll
-        for (int w = 0; w < kSoftmaxWarps; ++w) total += sums[w * HN + h];
-        l[h] = total;
-      }
-      const long long part0 = ((long long)p.sc.offsets[done.request] + done.chunk) * p.heads + head0;
-      if (done.chunks > 1 && threadIdx.x == 0) {
-#pragma unroll
-        for (int h = 0; h < HN; ++h)
-          if (head0 + h < p.heads) {
-            p.sc.part_m[part0 + h] = m[h];
-            p.sc.part_l[part0 + h] = l[h];
-          }
-      }
-      for (int d = 0; d < value_groups; ++d) {
+      score_sync();
+      for (int d = warp >> 2; d < value_groups; d += 2) {
         float v[HN], r[HN];
         tmem_load<HN>(tmem_o + d * 2 * HN + lane_addr, v);
         tmem_load<HN>(tmem_o + d * 2 * HN + HN + lane_addr, r);
-        const int c = d * 128 + warp * 32 + lane;
+        const int c = d * 128 + (warp & 3) * 32 + lane;
         if (c >= p.vdim) continue;
 #pragma unroll
         for (int h = 0; h < HN; ++h) {
           if (head0 + h >= p.heads) break;
+          const float x = (v[h] + r[h]) * factors[h];
           if (done.chunks == 1)
-            reinterpret_cast<T*>(p.out)[done.request * p.o_row + (head0 + h) * p.o_head + c] =
-                __float2bfloat16_rn((v[h] + r[h]) / fmaxf(l[h], 1.17549435e-38f));
+            reinterpret_cast<T*>(p.out)[done.request * p.o_row + (head0 + h) * p.o_head + c] = __float2bfloat16_rn(x);
           else
-            p.sc.part_o[(part0 + h) * p.vdim + c] = v[h] + r[h];
+            p.sc.part_o[(part0 + h) * p.vdim + c] = x;
         }
       }
       tc_fence_before();
       mbar_arrive(&bars[kOFree]);
-      softmax_sync();  // `sums` has been read before the next item's maxima reuse it
     }
     if (!ok && lane == 0) raise_status(p.status, MIE_STATUS_WAIT_TIMEOUT);
     // Requests with nothing to read (rejected metadata) get zeros.
-    for (int e = blockIdx.x * kSoftmaxWarps + warp; e < p.batch; e += gridDim.x * kSoftmaxWarps) {
+    for (int e = blockIdx.x * kScoreWarps + warp; e < p.batch; e += gridDim.x * kScoreWarps) {
       if (p.sc.offsets[e + 1] != p.sc.offsets[e]) continue;
       for (int h = 0; h < p.heads; ++h)
         for (int d = 2 * lane; d < p.vdim; d += 64)
@@ -439,27 +512,44 @@ __global__ void __launch_bounds__(kLatentThreads, 1)
   }
   tc_fence_before();
   __syncthreads();
-  if (warp == kSoftmaxWarps + 1) {
+  if (warp == kScoreWarps + 1) {
     tc_fence_after();
     tmem_dealloc(*tmem_slot, kTmemCols);
   }
 }
 
-template <int HN>
+template <int MT, int BOXES>
 int launch_latent(const CUtensorMap& map, LatentParams p, cudaStream_t stream) {
   p.ring = 2;
-  while (p.ring < kMaxRing && latent_layout(p.key_boxes, p.ring + 1, HN).total + 1024 <= 200 * 1024) ++p.ring;
-  const int smem = latent_layout(p.key_boxes, p.ring, HN).total + 1024;
+  while (p.ring < kMaxRing && latent_layout(p.key_boxes, p.ring + 1, MT).total + 1024 <= 224 * 1024) ++p.ring;
+  const int smem = latent_layout(p.key_boxes, p.ring, MT).total + 1024;
   static int configured[64] = {0};
   int dev = 0;
   MIE_CUDA(cudaGetDevice(&dev));
   if (dev < 0 || dev >= 64 || configured[dev] < smem) {
-    MIE_CUDA(cudaFuncSetAttribute(latent_decode_kernel<HN>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
+    MIE_CUDA(cudaFuncSetAttribute(latent_decode_kernel<MT, BOXES>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem));
     if (dev >= 0 && dev < 64) configured[dev] = smem;
   }
-  MIE_CUDA(launch_chained(latent_decode_kernel<HN>, dim3(sm_count()), dim3(kLatentThreads), (size_t)smem, stream, map, p));
+  MIE_CUDA(launch_chained(latent_decode_kernel<MT, BOXES>, dim3(sm_count()), dim3(kLatentThreads), (size_t)smem, stream,
+                          map, p));
   MIE_LAUNCH_CHECK("latent_decode_kernel");
   return MIE_OK;
+}
+
+template <int MT>
+int launch_latent_boxes(const CUtensorMap& map, const LatentParams& p, cudaStream_t stream) {
+  switch (p.key_boxes) {
+    case 1: return launch_latent<MT, 1>(map, p, stream);
+    case 2: return launch_latent<MT, 2>(map, p, stream);
+    case 3: return launch_latent<MT, 3>(map, p, stream);
+    case 4: return launch_latent<MT, 4>(map, p, stream);
+    case 5: return launch_latent<MT, 5>(map, p, stream);
+    case 6: return launch_latent<MT, 6>(map, p, stream);
+    case 7: return launch_latent<MT, 7>(map, p, stream);
+    case 8: return launch_latent<MT, 8>(map, p, stream);
+    case 9: return launch_latent<MT, 9>(map, p, stream);
+    default: return launch_latent<MT, kMaxKeyBoxes>(map, p, stream);
+  }
 }
 
 template <int VH>
@@ -537,7 +627,7 @@ extern "C" int mie_latent_decode_attention(const void* query, int64_t q_row_stri
                        IndexView(block_tables), IndexView(sequence_lengths), sc, batch, heads, block_size, num_blocks,
                        table_width, dim, value_dim, key_boxes, head_groups, 2, slab ? 1 : 0, scale * 1.4426950408889634f,
                        window, sinks, status};
-  if (int rc = item_heads == 16 ? launch_latent<16>(map, p, stream) : launch_latent<32>(map, p, stream)) return rc;
+  if (int rc = item_heads == 16 ? launch_latent_boxes<1>(map, p, stream) : launch_latent_boxes<2>(map, p, stream)) return rc;
   mie_view4_t q{const_cast<void*>(query), {q_row_stride, q_head_stride, 0, 1}};
   mie_view4_t o{out, {o_row_stride, o_head_stride, 0, 1}};
   const DecodeParams merge{View4(q), View4(o), p.tables, p.lengths, IndexView(), sc, batch, heads, 1, heads, block_size,
