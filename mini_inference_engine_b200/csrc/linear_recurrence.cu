@@ -470,8 +470,7 @@ __global__ void __launch_bounds__(256 * VD, KD + VD == 2 ? 2 : 1) outer_chunk_ke
       b *= whole;
     });
 #pragma unroll
-    for (int kt = 0; kt < 4; ++kt) {
-      if (kt * 16 >= n) break;
+    for (int kt = 0; kt < 4; ++kt) {  // k and v past the segment are zero
       uint32_t ka[4];
       const int unit = (s_row >> 3) + at_sel;  // 16-byte unit of the key row
       ldmatrix_x4_trans(ka[0], ka[1], ka[2], ka[3],
@@ -597,21 +596,6 @@ __device__ __forceinline__ void average_gates(float a, float u, float* keep, flo
   *add = gate * (u >= 0.f ? u + 0.5f : inv * da);
 }
 
-template <typename T, int VEC>
-struct AverageStep {
-  float zb[VEC], ub[VEC];
-  __device__ __forceinline__ AverageStep(const AverageParams& p, int c) {
-    Vec<T, VEC>::load(reinterpret_cast<const T*>(p.z_bias) + c, zb);
-    Vec<T, VEC>::load(reinterpret_cast<const T*>(p.u_bias) + c, ub);
-  }
-  __device__ __forceinline__ void gates(const float (&z)[VEC], const float (&u)[VEC], float (&keep)[VEC],
-                                        float (&add)[VEC]) const {
-#pragma unroll
-    for (int j = 0; j < VEC; ++j) average_gates(z[j] + zb[j], u[j] + ub[j], &keep[j], &add[j]);
-  }
-};
-constexpr int kAverageBatch = 4;  // tokens whose loads are in flight together
-
 // VEC activations as they lie in memory, widened when they are used.
 template <typename T, int VEC>
 struct alignas(sizeof(T) * VEC) RawVec {
@@ -621,7 +605,44 @@ struct alignas(sizeof(T) * VEC) RawVec {
 #pragma unroll
     for (int j = 0; j < VEC; ++j) out[j] = to_float<T>(v[j]);
   }
+  __device__ __forceinline__ static void load(const T* p, float (&out)[VEC]) { at(p).widen(out); }
+  __device__ __forceinline__ static void store(T* p, const float (&in)[VEC]) {
+    RawVec raw;
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) raw.v[j] = from_float<T>(in[j]);
+    *reinterpret_cast<RawVec*>(p) = raw;
+  }
 };
+
+template <>
+struct RawVec<__nv_bfloat16, 2> {  // one word, so that a batch of them costs one register each
+  uint32_t word;
+  __device__ __forceinline__ static RawVec at(const __nv_bfloat16* p) { return {*reinterpret_cast<const uint32_t*>(p)}; }
+  __device__ __forceinline__ void widen(float (&out)[2]) const {
+    out[0] = __uint_as_float(word << 16);
+    out[1] = __uint_as_float(word & 0xffff0000u);
+  }
+  __device__ __forceinline__ static void load(const __nv_bfloat16* p, float (&out)[2]) { at(p).widen(out); }
+  __device__ __forceinline__ static void store(__nv_bfloat16* p, const float (&in)[2]) {
+    *reinterpret_cast<uint32_t*>(p) = pack_bf16(in[0], in[1]);
+  }
+};
+
+template <typename T, int VEC>
+struct AverageStep {
+  float zb[VEC], ub[VEC];
+  __device__ __forceinline__ AverageStep(const AverageParams& p, int c) {
+    RawVec<T, VEC>::load(reinterpret_cast<const T*>(p.z_bias) + c, zb);
+    RawVec<T, VEC>::load(reinterpret_cast<const T*>(p.u_bias) + c, ub);
+  }
+  __device__ __forceinline__ void gates(const float (&z)[VEC], const float (&u)[VEC], float (&keep)[VEC],
+                                        float (&add)[VEC]) const {
+#pragma unroll
+    for (int j = 0; j < VEC; ++j) average_gates(z[j] + zb[j], u[j] + ub[j], &keep[j], &add[j]);
+  }
+};
+constexpr int kAverageBatch = 4;  // tokens loaded together, a batch ahead of the one that is computed
+
 
 // state * silu(g)
 template <typename T, int VEC>
@@ -629,7 +650,7 @@ __device__ __forceinline__ void average_emit(const float (&g)[VEC], T* out, cons
   float v[VEC];
 #pragma unroll
   for (int j = 0; j < VEC; ++j) v[j] = state[j] * silu(g[j]);
-  Vec<T, VEC>::store(out, v);
+  RawVec<T, VEC>::store(out, v);
 }
 
 template <typename T, int VEC>
@@ -643,25 +664,25 @@ __global__ void average_decode_kernel(AverageParams p) {
   const T* src = reinterpret_cast<const T*>(p.rows) + (long long)row * p.ld + c;
   const AverageStep<T, VEC> step(p, c);
   float state[VEC], keep[VEC], add[VEC], z[VEC], u[VEC], g[VEC];
-  Vec<T, VEC>::load(src, z);
-  Vec<T, VEC>::load(src + p.width, u);
-  Vec<T, VEC>::load(src + 2 * p.width, g);
+  RawVec<T, VEC>::load(src, z);
+  RawVec<T, VEC>::load(src + p.width, u);
+  RawVec<T, VEC>::load(src + 2 * p.width, g);
   if (p.positions.at(row) == 0) {
 #pragma unroll
     for (int j = 0; j < VEC; ++j) state[j] = 0.f;
   } else {
-    Vec<float, VEC>::load(slot + c, state);
+    RawVec<float, VEC>::load(slot + c, state);
   }
   step.gates(z, u, keep, add);
 #pragma unroll
   for (int j = 0; j < VEC; ++j) state[j] = keep[j] * state[j] + add[j];
-  Vec<float, VEC>::store(slot + c, state);
+  RawVec<float, VEC>::store(slot + c, state);
   average_emit<T, VEC>(g, reinterpret_cast<T*>(p.out) + (long long)row * p.ldo + c, state);
 }
 
 // What a segment does to a state before it: S -> product S + sum.
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128, 6) average_summary_kernel(AverageParams p) {
+__global__ void __launch_bounds__(128, 8) average_summary_kernel(AverageParams p) {
   chain_wait();
   chain_release();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
@@ -673,20 +694,24 @@ __global__ void __launch_bounds__(128, 6) average_summary_kernel(AverageParams p
   for (int j = 0; j < VEC; ++j) product[j] = 1.f, sum[j] = 0.f;
   const T* src = reinterpret_cast<const T*>(p.rows) + seg.begin * p.ld + c;
   const int count = (int)(seg.end - seg.begin);
-  for (int t0 = 0; t0 < count; t0 += kAverageBatch, src += kAverageBatch * p.ld) {
+  struct Batch {
     RawVec<T, VEC> z[kAverageBatch], u[kAverageBatch];
+  } batches[2];
+  auto fetch = [&](int t0, Batch& to) {
 #pragma unroll
     for (int i = 0; i < kAverageBatch; ++i)
       if (t0 + i < count) {
-        z[i] = RawVec<T, VEC>::at(src + i * p.ld);
-        u[i] = RawVec<T, VEC>::at(src + i * p.ld + p.width);
+        to.z[i] = RawVec<T, VEC>::at(src + (t0 + i) * p.ld);
+        to.u[i] = RawVec<T, VEC>::at(src + (t0 + i) * p.ld + p.width);
       }
+  };
+  auto advance = [&](int t0, const Batch& from) {
 #pragma unroll
     for (int i = 0; i < kAverageBatch; ++i) {
       if (t0 + i >= count) break;
       float keep[VEC], add[VEC], a[VEC], b[VEC];
-      z[i].widen(a);
-      u[i].widen(b);
+      from.z[i].widen(a);
+      from.u[i].widen(b);
       step.gates(a, b, keep, add);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) {
@@ -694,10 +719,17 @@ __global__ void __launch_bounds__(128, 6) average_summary_kernel(AverageParams p
         sum[j] = keep[j] * sum[j] + add[j];
       }
     }
+  };
+  fetch(0, batches[0]);
+  for (int t0 = 0; t0 < count; t0 += 2 * kAverageBatch) {
+    fetch(t0 + kAverageBatch, batches[1]);
+    advance(t0, batches[0]);
+    fetch(t0 + 2 * kAverageBatch, batches[0]);
+    advance(t0 + kAverageBatch, batches[1]);
   }
   float* dst = p.carry + (long long)blockIdx.x * 2 * p.width + c;
-  Vec<float, VEC>::store(dst, product);
-  Vec<float, VEC>::store(dst + p.width, sum);
+  RawVec<float, VEC>::store(dst, product);
+  RawVec<float, VEC>::store(dst + p.width, sum);
 }
 
 // carry[segment][0] <- state before the segment.
@@ -736,7 +768,7 @@ __global__ void average_carry_kernel(AverageParams p) {
 }
 
 template <typename T, int VEC>
-__global__ void __launch_bounds__(128, 6) average_segment_kernel(AverageParams p) {
+__global__ void __launch_bounds__(128, 8) average_segment_kernel(AverageParams p) {
   chain_wait();
   chain_release();
   const int c = (blockIdx.y * blockDim.x + threadIdx.x) * VEC;
@@ -747,39 +779,50 @@ __global__ void __launch_bounds__(128, 6) average_segment_kernel(AverageParams p
   const AverageStep<T, VEC> step(p, c);
   float state[VEC];
   if (p.carry != nullptr) {
-    Vec<float, VEC>::load(p.carry + (long long)blockIdx.x * 2 * p.width + c, state);
+    RawVec<float, VEC>::load(p.carry + (long long)blockIdx.x * 2 * p.width + c, state);
   } else if (p.positions.at(seg.begin) == 0) {
 #pragma unroll
     for (int j = 0; j < VEC; ++j) state[j] = 0.f;
   } else {
-    Vec<float, VEC>::load(slot + c, state);
+    RawVec<float, VEC>::load(slot + c, state);
   }
   const T* src = reinterpret_cast<const T*>(p.rows) + seg.begin * p.ld + c;
   T* out = reinterpret_cast<T*>(p.out) + seg.begin * p.ldo + c;
   const int count = (int)(seg.end - seg.begin);
-  for (int t0 = 0; t0 < count; t0 += kAverageBatch, src += kAverageBatch * p.ld, out += kAverageBatch * p.ldo) {
+  struct Batch {
     RawVec<T, VEC> z[kAverageBatch], u[kAverageBatch], g[kAverageBatch];
+  } batches[2];
+  auto fetch = [&](int t0, Batch& to) {
 #pragma unroll
     for (int i = 0; i < kAverageBatch; ++i)
       if (t0 + i < count) {
-        z[i] = RawVec<T, VEC>::at(src + i * p.ld);
-        u[i] = RawVec<T, VEC>::at(src + i * p.ld + p.width);
-        g[i] = RawVec<T, VEC>::at(src + i * p.ld + 2 * p.width);
+        to.z[i] = RawVec<T, VEC>::at(src + (t0 + i) * p.ld);
+        to.u[i] = RawVec<T, VEC>::at(src + (t0 + i) * p.ld + p.width);
+        to.g[i] = RawVec<T, VEC>::at(src + (t0 + i) * p.ld + 2 * p.width);
       }
+  };
+  auto advance = [&](int t0, const Batch& from) {
 #pragma unroll
     for (int i = 0; i < kAverageBatch; ++i) {
       if (t0 + i >= count) break;
       float keep[VEC], add[VEC], a[VEC], b[VEC];
-      z[i].widen(a);
-      u[i].widen(b);
+      from.z[i].widen(a);
+      from.u[i].widen(b);
       step.gates(a, b, keep, add);
 #pragma unroll
       for (int j = 0; j < VEC; ++j) state[j] = keep[j] * state[j] + add[j];
-      g[i].widen(a);
-      average_emit<T, VEC>(a, out + i * p.ldo, state);
+      from.g[i].widen(a);
+      average_emit<T, VEC>(a, out + (t0 + i) * p.ldo, state);
     }
+  };
+  fetch(0, batches[0]);
+  for (int t0 = 0; t0 < count; t0 += 2 * kAverageBatch) {
+    fetch(t0 + kAverageBatch, batches[1]);
+    advance(t0, batches[0]);
+    fetch(t0 + 2 * kAverageBatch, batches[0]);
+    advance(t0 + kAverageBatch, batches[1]);
   }
-  if (seg.last) Vec<float, VEC>::store(slot + c, state);
+  if (seg.last) RawVec<float, VEC>::store(slot + c, state);
 }
 
 // ---------------------------------------------------------------------------
@@ -961,13 +1004,13 @@ extern "C" int mie_gated_average(const void* rows, int64_t ld, const void* z_bia
     p.seg.length = segment_tokens;
     p.carry = carry;
   }
-  const int act = dtype == MIE_DTYPE_BF16 ? 8 : 16;
-  const bool vec = width % 4 == 0 && ld % 4 == 0 && ldo % 4 == 0 && slot_stride % 4 == 0 && aligned(rows, act) &&
-                   aligned(z_bias, act) && aligned(u_bias, act) && aligned(out, act) && aligned(state, 16) &&
-                   aligned(carry, 16);
+  const int act = dtype == MIE_DTYPE_BF16 ? 4 : 8;  // bytes of two activations
+  const bool vec = width % 2 == 0 && ld % 2 == 0 && ldo % 2 == 0 && slot_stride % 2 == 0 && aligned(rows, act) &&
+                   aligned(z_bias, act) && aligned(u_bias, act) && aligned(out, act) && aligned(state, 8) &&
+                   aligned(carry, 8);
   if (dtype == MIE_DTYPE_BF16)
-    return vec ? launch_average<__nv_bfloat16, 4>(p, decode, segments, stream)
+    return vec ? launch_average<__nv_bfloat16, 2>(p, decode, segments, stream)
                : launch_average<__nv_bfloat16, 1>(p, decode, segments, stream);
-  return vec ? launch_average<float, 4>(p, decode, segments, stream)
+  return vec ? launch_average<float, 2>(p, decode, segments, stream)
              : launch_average<float, 1>(p, decode, segments, stream);
 }

@@ -29,6 +29,7 @@ from mini_inference_engine_b200.engine.kernels.recurrence import gated_average, 
 from mini_inference_engine_b200.engine.kv_cache.latent_attention import (
     VisibleSpans,
     latent_decode_attention,
+    latent_decode_scratch,
     latent_norm_write,
     rotate_heads,
 )
@@ -373,9 +374,20 @@ def _ripesun_kernels(size, ripe: RipesunRunner, tide: TidelornRunner, batch, con
     t_key = tide._attention[0][0]
     common = dict(window=window, status=ripe.status)
 
-    def t_decode():
+    def planned(attend):
+        """Calls that use the step's work plan, as every layer of a geometry but the first does."""
+
+        attend(False, 0)
+        slots_used = iter(range(1, 64))
+        return lambda: attend(True, next(slots_used))
+
+    def t_attend(plan, slot):
         sink_decode_attention(t_query[:batch], t_out[:batch], tide.key_blocks[0], tide.value_blocks[0], tables, lengths,
-                              scale=0.1, sinks=t.sinks, scratch=tide._scratch[t_key], **common)
+                              scale=0.1, sinks=t.sinks, scratch=tide._scratch[t_key], use_plan=plan, plan_slot=slot, **common)
+
+    def attend(pool, tab, lens, window, scratch):
+        return lambda plan, slot: latent_decode_attention(query, latent_out, pool, tab, lens, scale=0.1, sinks=w.sinks,
+                                                          window=window, scratch=scratch, use_plan=plan, status=ripe.status)
 
     def t_prefill():
         sink_prefill_attention(t_query, t_out, tide.key_blocks[0], tide.value_blocks[0], tables_p, cu, lens,
@@ -383,11 +395,19 @@ def _ripesun_kernels(size, ripe: RipesunRunner, tide: TidelornRunner, batch, con
 
     t_decode_work = {"bytes_": batch * reach * kv * t_dim * 4}
     t_prefill_work = {"flops": 4 * t_heads * t_dim * inside}
-    pair("decode attention", lambda: latent_decode_attention(
-        query, latent_out, ripe.latents[0], tables, lengths, scale=0.1, sinks=w.sinks,
-        scratch=ripe._scratch[ripe._streams[0][0]], **common), t_decode,
-        work={"bytes_": batch * reach * mixer.row * 2, "flops": 2 * heads * batch * reach * (mixer.row + KV_RANK)},
-        their_work=t_decode_work)
+    def latent_work(seen):
+        return {"bytes_": batch * seen * mixer.row * 2, "flops": 2 * heads * batch * seen * (mixer.row + KV_RANK)}
+
+    pair("decode attention", planned(attend(ripe.latents[0], tables, lengths, window, ripe._scratch[ripe._streams[0][0]])),
+         planned(t_attend), work=latent_work(reach), their_work=t_decode_work)
+    # The same bytes as the other design's window: a cached row is that much smaller.
+    equal = t_decode_work["bytes_"] // (batch * mixer.row * 2)
+    deep = torch.randn(batch * -(-equal // page), 1, page, mixer.row, device=device).to(torch.bfloat16)
+    pair("decode attention, equal bytes", planned(attend(
+        deep, _tables(batch, -(-equal // page), deep.shape[0], device), torch.full_like(lengths, equal), None,
+        latent_decode_scratch(batch, heads, KV_RANK, batch * equal, device))), planned(t_attend),
+        work=latent_work(equal), their_work=t_decode_work)
+    del deep
     spans = VisibleSpans(cu, lens, window=window, tokens=tokens, max_query_len=prompt_len, max_context=prompt_len,
                          chunk_starts=[0] * prompts, status=ripe.status)
     rows = spans.gather(ripe.latents[0], tables_p)
@@ -410,13 +430,13 @@ def _ripesun_kernels(size, ripe: RipesunRunner, tide: TidelornRunner, batch, con
     # Recurrent mixers beside attention, then everything that is a pass over rows, then products.
     for label, n, pos, own, tab in (("decode", batch, lengths - 1, None, tables), ("prefill", tokens, flat, owners, tables_p)):
         chunk = {} if label == "decode" else {"cu_seqlens": cu, "max_query_len": prompt_len}
-        attend, attend_work = (t_decode, t_decode_work) if label == "decode" else (t_prefill, t_prefill_work)
+        t_mix, attend_work = (planned(t_attend), t_decode_work) if label == "decode" else (t_prefill, t_prefill_work)
         requests = batch if label == "decode" else prompts
         state_bytes = 4 * (2 if label == "decode" else 1) * requests  # chunks that start at position 0 only write it
         o_rows, o_out = bf16(n, outer.inputs.shape[0]), bf16(n, values)
         pair(f"{label} outer recurrence", lambda: outer_recurrence(
             o_rows, o_out, outer.decay, ripe.state.layer(0), slots[:requests], pos, heads=heads, dim=HEAD, value_dim=HEAD,
-            status=ripe.status, **chunk), attend,
+            status=ripe.status, **chunk), t_mix,
             work={"bytes_": state_bytes * heads * HEAD * HEAD + 2 * n * 4 * values}, their_work=attend_work)
         a_rows, a_out = bf16(n, 3 * width), bf16(n, width)
         t_act = bf16(n, 2 * ff)
