@@ -95,8 +95,8 @@ def test_random_weights_have_the_checkpoint_form():
 
 
 def test_segments_are_cut_only_when_lanes_are_few():
-    assert segment_tokens(200, 1) == 0 and segment_tokens(5000, 148) == 0
-    assert segment_tokens(300, 4) == 256 and segment_tokens(8192, 16) == 448
+    assert segment_tokens(200, 1) == 0 and segment_tokens(5000, 75) == 0
+    assert segment_tokens(300, 4) == 256 and segment_tokens(8192, 16) == 960
     assert segment_tokens(1 << 20, 64, sm_count=148) % 64 == 0
 
 
