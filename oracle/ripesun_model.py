@@ -81,7 +81,7 @@ def decayed_outer_products(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, de
 
 
 def gru_candidate(u: torch.Tensor) -> torch.Tensor:
-    """u + 1/2 where u >= 0, sigmoid(u) elsewhere."""
+    """Half a unit above u on the non-negative side, the logistic function on the negative one (both 1/2 at 0)."""
 
     return torch.where(u >= 0, u + 0.5, torch.sigmoid(u))
 
